@@ -30,6 +30,9 @@ __all__ = [
     "matmul",
     "linear",
     "linear_residual",
+    "linear_wide",
+    "residual_norm",
+    "softcap",
     "rms_norm",
     "rope",
     "swiglu",
@@ -102,8 +105,33 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
             pad = (-n) % 8
             y = _cuda.linear(x, F.pad(weight, (0, 0, 0, pad)), None if bias is None else F.pad(bias, (0, pad)))
             return y[..., :n]
-        _fallback("linear", f"K={x.shape[-1]} is not a multiple of 8 (TMA row pitch)", x)
+        # a contraction width that is not a multiple of 8 (TMA row pitch): zero columns on both operands add nothing
+        pad = (-x.shape[-1]) % 8
+        return linear(F.pad(x, (0, pad)), F.pad(weight, (0, pad)), bias)
     return F.linear(x, weight, bias)
+
+
+def linear_wide(x: torch.Tensor, weight: torch.Tensor) -> torch.Tensor:
+    """``x @ weight.T`` with an fp32 result: the bf16 tensor-core accumulators are stored unrounded (inference; vocabulary logits)."""
+    if _native(x) and weight.dtype == torch.bfloat16 and not (torch.is_grad_enabled() and (x.requires_grad or weight.requires_grad)):
+        from . import _cuda
+
+        n, pad_k, pad_n = weight.shape[0], (-x.shape[-1]) % 8, (-weight.shape[0]) % 8
+        if pad_k or pad_n:
+            x, weight = F.pad(x, (0, pad_k)), F.pad(weight, (0, pad_k, 0, pad_n))
+        y = _cuda.gemm(x.reshape(-1, x.shape[-1]), weight, out_dtype=torch.float32)
+        return y[:, :n].reshape(*x.shape[:-1], n)
+    return linear(x, weight).float()
+
+
+def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    """``cap · tanh(logits / cap)``; fp32 CUDA logits outside autograd are capped in place in one pass."""
+    if _native(logits, (torch.float32,)) and logits.is_contiguous() and logits.numel() > 0 and not (torch.is_grad_enabled() and logits.requires_grad):
+        from ._lib import check, lib, stream_ptr
+
+        check(lib().ttb_softcap(logits.data_ptr(), logits.numel(), float(cap), stream_ptr()), "softcap")
+        return logits
+    return torch.tanh(logits / cap) * cap
 
 
 def linear_residual(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], residual: torch.Tensor) -> torch.Tensor:
@@ -200,6 +228,20 @@ def rms_norm(x: torch.Tensor, scale: Optional[torch.Tensor], eps: float = 1e-6) 
     return reference.rms_norm(x, scale, eps)
 
 
+def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor], w_next: Optional[torch.Tensor], *, eps: float, mult: float = 1.0,
+                  offset: float = 0.0) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """The step between two sublayers on a 32-bit residual stream ``x``: ``x' = x + mult · norm(y; w_post)`` (``y=None``: ``x' = x``)
+    and ``h = norm(x'; w_next)`` in the gain's dtype (``w_next=None``: no ``h``), with ``norm(z; w) = z / rms(z) · (offset + w)`` in
+    fp32.  Returns ``(x', h)``."""
+    grads = torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in (x, y, w_post, w_next))
+    w = w_post if w_post is not None else w_next
+    if cuda_ops_enabled(x) and x.dtype == torch.float32 and not grads and w.dtype in (torch.bfloat16, torch.float32) and (y is None or y.dtype == w.dtype) and x.numel() > 0:
+        from . import latent
+
+        return latent.residual_norm(x, y, w_post, w_next, eps, mult, offset)
+    return reference.residual_norm(x, y, w_post, w_next, eps=eps, mult=mult, offset=offset)
+
+
 def rope(
     x: torch.Tensor, cache: torch.Tensor, input_pos: Optional[torch.Tensor] = None, interleaved: bool = True
 ) -> torch.Tensor:
@@ -238,6 +280,8 @@ def attention(
         why = None
         if dropout_p != 0.0:
             why = "attention dropout"
+        elif mask.key_start is not None and (mask.doc_ids is not None or mask.chunk > 0 or mask.window > 0 or mask.bool_mask is not None):
+            why = "key_start together with another mask kind"
         elif q.shape[-1] not in (64, 128):
             why = f"head_dim {q.shape[-1]}"
         else:
@@ -245,6 +289,8 @@ def attention(
         if why is None:
             return _cuda_attention.attention(q, k, v, mask, scale, softcap)
         _fallback("attention", why, q)
+    if mask.key_start is not None:
+        mask = AttentionMask(causal=False, bool_mask=mask.dense(q.shape[0], q.shape[1], k.shape[1], q.device))
     return reference.attention(
         q,
         k,

@@ -132,7 +132,13 @@ def attention(q, k, v, mask: AttentionMask, scale: Optional[float], softcap: flo
     scale = (1.0 / math.sqrt(d)) if scale is None else scale
     lo = hi = kmask = None
     monotone, causal = 1, bool(mask.causal)
-    if mask.bool_mask is not None:
+    if mask.key_start is not None:
+        if mask.key_start.numel() != b or mask.query_start + s > sk:
+            raise ValueError("key_start / query_start do not fit the query and key lengths")
+        lo = mask.key_start.to(device=q.device, dtype=torch.int32).view(b, 1).expand(b, s).contiguous()
+        hi = (torch.arange(s, device=q.device, dtype=torch.int32) + mask.query_start).view(1, s).expand(b, s).contiguous()
+        causal = False
+    elif mask.bool_mask is not None:
         cached = getattr(mask, "_dense_cache", None)
         if cached is not None and cached[0] == (b, s, sk, mask.bool_mask.data_ptr()):
             kmask, lo, hi = cached[1]

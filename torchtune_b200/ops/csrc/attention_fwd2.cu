@@ -11,19 +11,17 @@
 // Masks: per-query bounds lo / hi that do not decrease along the sequence (causal, packed documents, sliding windows, chunks), or
 // none.  Each tile visits only its own range of key blocks.  Element-wise masks, soft-capping and head dims other than 128 stay on
 // the one-tile kernel in attention.cu.  Every wait is bounded and reports through the error word.
+#include "common/attn_math.cuh"
 #include "common/ptx.cuh"
 #include "common/tmap.h"
 
 namespace ttb {
 namespace fa2 {
 
-static constexpr int kBlk = 128;
+using namespace attn;
 static constexpr int D = 128;
-static constexpr int kPanelBytes = 16384;  // 128 rows x 128 B (64 bf16 columns)
 static constexpr int kTileBytes = kBlk * D * 2;
 static constexpr int kThreads = 384;
-static constexpr float kLog2e = 1.4426950408889634f;
-static constexpr float kRescaleThreshold = 8.0f;  // log2 units
 static constexpr int kSmemBytes = 6 * kTileBytes + 1024 + 256;
 
 struct Params {
@@ -36,45 +34,6 @@ struct Params {
   float* lse;
   int* err;
 };
-
-__device__ __forceinline__ uint64_t desc_kmajor(uint32_t base, int k) {
-  return make_smem_desc_sw128(base + (k >> 2) * kPanelBytes + (k & 3) * 32, 16, 1024);
-}
-__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t base, int k) {
-  return make_smem_desc_sw128(base + k * 2048, kPanelBytes, 1024);
-}
-__device__ __forceinline__ float max3(float a, float b, float c) {
-  float d;
-  asm("max.f32 %0, %1, %2, %3;" : "=f"(d) : "f"(a), "f"(b), "f"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t pack_f32x2(float lo, float hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "f"(lo), "f"(hi));
-  return d;
-}
-__device__ __forceinline__ uint64_t pack_u32x2(uint32_t lo, uint32_t hi) {
-  uint64_t d;
-  asm("mov.b64 %0, {%1, %2};" : "=l"(d) : "r"(lo), "r"(hi));
-  return d;
-}
-__device__ __forceinline__ void unpack_f32x2(uint64_t v, float& lo, float& hi) {
-  asm("mov.b64 {%0, %1}, %2;" : "=f"(lo), "=f"(hi) : "l"(v));
-}
-__device__ __forceinline__ uint64_t fma_f32x2(uint64_t a, uint64_t b, uint64_t c) {
-  uint64_t d;
-  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-  return d;
-}
-__device__ __forceinline__ uint64_t add_f32x2(uint64_t a, uint64_t b) {
-  uint64_t d;
-  asm("add.rn.f32x2 %0, %1, %2;" : "=l"(d) : "l"(a), "l"(b));
-  return d;
-}
-__device__ __forceinline__ void fail(volatile int* abort_flag, int* err, int code) {
-  *abort_flag = 1;
-  atomicExch(err, code);
-}
 
 __global__ void __launch_bounds__(kThreads, 1)
 attn_fwd2_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, Params p) {

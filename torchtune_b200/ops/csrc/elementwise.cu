@@ -328,6 +328,12 @@ __global__ void swiglu_bwd_kernel(const __nv_bfloat16* __restrict__ dy, const __
   }
 }
 
+// x <- cap * tanh(x / cap), fp32 in place.
+__global__ void softcap_kernel(float* __restrict__ x, long long n, float cap) {
+  for (long long i = blockIdx.x * static_cast<long long>(blockDim.x) + threadIdx.x; i < n; i += static_cast<long long>(gridDim.x) * blockDim.x)
+    x[i] = tanhf(x[i] / cap) * cap;
+}
+
 static inline int grid_for(long long work_items, int threads) {
   long long blocks = (work_items + threads - 1) / threads;
   const long long cap = static_cast<long long>(sm_count()) * 16;
@@ -432,6 +438,13 @@ extern "C" int ttb_swiglu_fwd(const void* g, const void* u, void* y, long long r
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 
+extern "C" int ttb_softcap(float* x, long long n, float cap, void* stream) {
+  if (n <= 0 || !(cap > 0.f)) return kErrBadShape;
+  TTB_COUNT_LAUNCH(1);
+  softcap_kernel<<<grid_for(n, 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(x, n, cap);
+  return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
+}
+
 extern "C" int ttb_swiglu_bwd(const void* dy, const void* g, const void* u, void* dg, void* du, long long rows, int H,
                               long long lddy, long long ldg, long long ldu, long long lddg, long long lddu,
                               void* stream) {
@@ -511,8 +524,9 @@ extern "C" int ttb_rmsnorm_bwd_noalloc(const void* dy, const void* x, const void
 
 extern "C" unsigned int ttb_violations_embedding(int reset);
 extern "C" unsigned int ttb_violations_loss(int reset);
+extern "C" unsigned int ttb_violations_latent(int reset);
 
 // Out-of-range user indices (token ids, labels, positions) that kernels replaced by a safe value since the last reset.
 extern "C" unsigned int ttb_index_violations(int reset) {
-  return ttb_violations_rope(reset) + ttb_violations_embedding(reset) + ttb_violations_loss(reset);
+  return ttb_violations_rope(reset) + ttb_violations_embedding(reset) + ttb_violations_loss(reset) + ttb_violations_latent(reset);
 }

@@ -22,12 +22,16 @@ class AttentionMask:
     chunk: int = 0  # >0: positions attend only inside the same chunk of this size
     window: int = 0  # >0: key must be within this many positions before the query
     bool_mask: Optional[torch.Tensor] = None  # dense [b, sq, skv], True = attend
+    # Cached decoding of left-padded rows: query i sits in cache slot query_start + i and sees the slots key_start[b] ... its own.
+    key_start: Optional[torch.Tensor] = None  # [b] int32
+    query_start: int = 0
 
     def to(self, device, non_blocking: bool = False) -> "AttentionMask":
         return replace(
             self,
             doc_ids=None if self.doc_ids is None else self.doc_ids.to(device, non_blocking=non_blocking),
             bool_mask=None if self.bool_mask is None else self.bool_mask.to(device, non_blocking=non_blocking),
+            key_start=None if self.key_start is None else self.key_start.to(device, non_blocking=non_blocking),
         )
 
     def with_chunk(self, chunk: int) -> "AttentionMask":
@@ -39,6 +43,13 @@ class AttentionMask:
             return self.bool_mask
         from .reference import dense_mask
 
+        if self.key_start is not None:
+            j = torch.arange(skv, device=device)
+            own = self.query_start + torch.arange(sq, device=device)
+            m = (j[None, None, :] <= own[None, :, None]) & (j[None, None, :] >= self.key_start.to(device)[:, None, None])
+            if self.doc_ids is not None or self.chunk > 0 or self.window > 0:
+                raise ValueError("key_start does not combine with document ids, chunks or windows")
+            return m.expand(b, sq, skv)
         m = dense_mask(b, sq, skv, device, self.causal, self.doc_ids, self.chunk, self.window)
         return None if m is None else m.squeeze(1)
 

@@ -22,6 +22,31 @@ def rms_norm(x: torch.Tensor, scale: Optional[torch.Tensor], eps: float) -> torc
     return y if scale is None else y * scale
 
 
+def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[torch.Tensor], w_next: Optional[torch.Tensor], *, eps: float, mult: float,
+                  offset: float) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """``x' = x + mult · norm(y; w_post)``, ``h = norm(x'; w_next)`` with ``norm(z; w) = z / sqrt(mean(z²) + eps) · (offset + w)``, all in
+    fp32; ``x'`` is fp32, ``h`` has the gain's dtype."""
+
+    def norm(z: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+        zf = z.float()
+        return zf * torch.rsqrt(zf.pow(2).mean(-1, keepdim=True) + eps) * (offset + w.float())
+
+    x = x.float()
+    if y is not None:
+        x = x + mult * norm(y, w_post)
+    return x, None if w_next is None else norm(x, w_next).to(w_next.dtype)
+
+
+def latent_attention(q: torch.Tensor, k_up: torch.Tensor, k_rot: torch.Tensor, v: torch.Tensor, visible: torch.Tensor, scale: float) -> torch.Tensor:
+    """Attention with a key part shared by all heads: ``q`` ``[b, s, h, d + r]``, ``k_up`` ``[b, sk, h, d]``, ``k_rot`` ``[b, sk, r]``, ``v``
+    ``[b, sk, h, dv]``, ``visible`` ``[b | 1, s, sk]``.  Scores and weights in fp32; a row without keys gives 0."""
+    d = k_up.shape[-1]
+    qf = q.float()
+    s = (torch.einsum("bqhd,bkhd->bhqk", qf[..., :d], k_up.float()) + torch.einsum("bqhr,bkr->bhqk", qf[..., d:], k_rot.float())) * scale
+    p = torch.nan_to_num(torch.softmax(s.masked_fill(~visible.unsqueeze(1), float("-inf")), dim=-1), nan=0.0)
+    return torch.einsum("bhqk,bkhd->bqhd", p, v.float()).to(q.dtype)
+
+
 def rope_interleaved(x: torch.Tensor, cache: torch.Tensor, input_pos: Optional[torch.Tensor]) -> torch.Tensor:
     """Rotate pairs ``(x[2i], x[2i+1])``; ``x`` is ``[b, s, h, d]``, ``cache`` is
     ``[max_seq, d/2, 2]`` of (cos, sin) (torchtune/modules/position_embeddings.py:69-122)."""
