@@ -19,8 +19,10 @@ from torch import nn
 from ..modules import (
     FeedForward,
     FrozenNF4Linear,
+    LatentAttention,
     Linear,
     MultiHeadAttention,
+    ResidualStreamLayer,
     RMSNorm,
     TiedLinear,
     TransformerDecoder,
@@ -91,6 +93,12 @@ class DecoderArch:
     mlp_factory: Optional[Callable[[int, "AdapterSpec"], nn.Module]] = None
     layer_uses_rope: Optional[Callable[[int], bool]] = None
     layer_mask_mod: Optional[Callable[[int], Optional[Callable]]] = None
+    attn_factory: Optional[Callable[[int, "AdapterSpec"], nn.Module]] = None
+    # 32-bit residual stream with a norm on both sides of every sublayer (post_norms), whose outputs enter multiplied by residual_mult;
+    # `mlp_factory` may return None for a layer without a feed-forward block
+    residual_stream: bool = False
+    residual_mult: float = 1.0
+    wide_logits: bool = False
 
     def resolved_head_dim(self) -> int:
         return self.head_dim or self.embed_dim // self.num_heads
@@ -167,9 +175,15 @@ def build_decoder(arch: DecoderArch, adapter: Optional[AdapterSpec] = None) -> T
         if arch.layer_mask_mod is not None and mask_mod is None:
             mask_mod = arch.layer_mask_mod(idx)
         mlp = arch.mlp_factory(idx, ad) if arch.mlp_factory else build_mlp(arch.embed_dim, arch.resolved_hidden(), ad, arch.activation(), arch.mlp_bias)
+        attn = arch.attn_factory(idx, ad) if arch.attn_factory else build_attention(arch, ad, rope, positional)
+        if arch.residual_stream:
+            norm = lambda: arch.norm(arch.embed_dim, arch.norm_eps)  # noqa: E731
+            layers.append(ResidualStreamLayer(attn, mlp, sa_norm=norm(), sa_scale=norm(), mlp_norm=norm() if mlp is not None else None,
+                                              mlp_scale=norm() if mlp is not None else None, residual_mult=arch.residual_mult))
+            continue
         layers.append(
             TransformerSelfAttentionLayer(
-                attn=build_attention(arch, ad, rope, positional),
+                attn=attn,
                 mlp=mlp,
                 sa_norm=arch.norm(arch.embed_dim, arch.norm_eps),
                 mlp_norm=arch.norm(arch.embed_dim, arch.norm_eps),
@@ -199,6 +213,8 @@ def build_decoder(arch: DecoderArch, adapter: Optional[AdapterSpec] = None) -> T
         output=output,
     )
     model.logit_softcap = float(arch.logit_softcap)
+    model.wide_logits = bool(arch.wide_logits)
+    model.span_masks = all(isinstance(layer.attn, LatentAttention) for layer in layers)
     if ad.quantize_base:
         # checkpoints of a quantised-base model are written in bf16 on CPU
         _register_reparametrize_state_dict_hooks(model, dtype=tok.weight.dtype)

@@ -11,6 +11,7 @@ from .common_utils import (
 from .embedding_utils import resize_token_embeddings
 from .feed_forward import FeedForward
 from .kv_cache import KVCache
+from .latent_attention import LatentAttention, LatentCache
 from .layer_norm import Fp32LayerNorm
 from .linear import Linear
 from .low_precision import FrozenNF4Linear
@@ -23,10 +24,10 @@ from .position_embeddings import (
     RotaryPositionalEmbeddings,
     VisionRotaryPositionalEmbeddings,
 )
-from .rms_norm import RMSNorm, rms_norm
+from .rms_norm import RMSNorm, StreamRMSNorm, rms_norm
 from .tanh_gate import TanhGate
 from .tied_linear import TiedLinear
-from .transformer import TransformerCrossAttentionLayer, TransformerDecoder, TransformerSelfAttentionLayer
+from .transformer import ResidualStreamLayer, TransformerCrossAttentionLayer, TransformerDecoder, TransformerSelfAttentionLayer
 from .layer_dropout import LayerDropout, ModuleLayerDropoutWrapper, ScaleType, get_scale, prepare_layer_dropout
 from .vq_embeddings import VectorQuantizedEmbeddings
 from .vision_transformer import CLSEmbedding, CLSProjection, PatchEmbedding, VisionTransformer
@@ -49,6 +50,8 @@ __all__ = [
     "FeedForward",
     "FrozenNF4Linear",
     "KVCache",
+    "LatentAttention",
+    "LatentCache",
     "Linear",
     "RotaryPositionalEmbeddings",
     "VisionRotaryPositionalEmbeddings",
@@ -58,11 +61,13 @@ __all__ = [
     "Qwen2RotaryPositionalEmbeddings",
     "Phi3RotaryPositionalEmbeddings",
     "RMSNorm",
+    "StreamRMSNorm",
     "rms_norm",
     "TiedLinear",
     "Fp32LayerNorm",
     "TransformerDecoder",
     "TransformerSelfAttentionLayer",
+    "ResidualStreamLayer",
     "TransformerCrossAttentionLayer",
     "reparametrize_as_dtype_state_dict_post_hook",
     "delete_kv_caches",

@@ -58,8 +58,9 @@ def slice_str_to_array(slice_str: str, length: int) -> List[bool]:
 
 def _attention_modules(model: nn.Module):
     from .attention import MultiHeadAttention
+    from .latent_attention import LatentAttention
 
-    return [m for m in model.modules() if isinstance(m, MultiHeadAttention)]
+    return [m for m in model.modules() if isinstance(m, (MultiHeadAttention, LatentAttention))]
 
 
 @contextlib.contextmanager

@@ -10,6 +10,7 @@ from torch import nn
 from .. import ops
 from ..ops.mask import AttentionMask
 from .attention import MaskLike, MultiHeadAttention
+from .rms_norm import StreamRMSNorm
 
 
 class TransformerSelfAttentionLayer(nn.Module):
@@ -74,6 +75,35 @@ class TransformerSelfAttentionLayer(nn.Module):
         if self._fuse_residual_mlp:
             return self.mlp(self.mlp_norm(h), residual=h)
         return h + self.mlp_scale(self.mlp(self.mlp_norm(h)))
+
+
+class ResidualStreamLayer(TransformerSelfAttentionLayer):
+    """Decoder layer on a 32-bit residual stream with a norm on both sides of each sublayer:
+    ``x = x + m · sa_scale(attn(sa_norm(x)))``, then ``x = x + m · mlp_scale(mlp(mlp_norm(x)))`` (left out with ``mlp=None``).
+
+    All four norms are :class:`~torchtune_b200.modules.StreamRMSNorm`, so the end of one sublayer and the norm in front of the next run
+    as one pass over the stream.  A decoder that chains layers passes ``(x, sa_norm(x))`` and the norm that follows this layer, and
+    receives the same kind of pair for the next one."""
+
+    def __init__(self, attn: nn.Module, mlp: Optional[nn.Module], *, sa_norm: nn.Module, sa_scale: nn.Module, mlp_norm: Optional[nn.Module] = None, mlp_scale: Optional[nn.Module] = None,
+                 residual_mult: float = 1.0) -> None:
+        nn.Module.__init__(self)
+        if (mlp is None) != (mlp_norm is None) or (mlp is None) != (mlp_scale is None):
+            raise ValueError("the feed-forward block and its two norms come together")
+        self.attn, self.mlp = attn, mlp
+        self.sa_norm, self.sa_scale, self.mlp_norm, self.mlp_scale = sa_norm, sa_scale, mlp_norm, mlp_scale
+        self.mask_mod = None
+        self.residual_mult = float(residual_mult)
+
+    def forward(self, x, *, mask: MaskLike = None, input_pos: Optional[torch.Tensor] = None, layer_state: Optional[dict] = None, next_norm: Optional[nn.Module] = None, **kwargs):
+        x, normed = x if isinstance(x, tuple) else (x.float(), None)
+        if normed is None:
+            normed = self.sa_norm(x)
+        chain, m = StreamRMSNorm.chain, self.residual_mult
+        x, normed = chain(x, self.attn(normed, mask=mask, input_pos=input_pos, layer_state=layer_state), self.sa_scale, m, next_norm if self.mlp is None else self.mlp_norm)
+        if self.mlp is not None:
+            x, normed = chain(x, self.mlp(normed), self.mlp_scale, m, next_norm)
+        return x if next_norm is None else (x, normed)
 
 
 class TransformerCrossAttentionLayer(nn.Module):
@@ -199,6 +229,10 @@ class TransformerDecoder(nn.Module):
         # cap·tanh(logits/cap) applied to the logits (Gemma-2); 0 = none.  A loss that takes the hidden states instead
         # (``skip_output_layer``) reads this attribute and applies the cap itself.
         self.logit_softcap = 0.0
+        # Vocabulary logits leave the output projection in fp32 instead of being widened from its rounded result.
+        self.wide_logits = False
+        # Prompts of unequal length may be described to the layers by the first key of every row instead of a boolean mask.
+        self.span_masks = False
         self.encoder_max_cache_seq_len = None
         self.decoder_max_cache_seq_len = None
 
@@ -245,7 +279,7 @@ class TransformerDecoder(nn.Module):
     # -- forward ---------------------------------------------------------------
     def _cap(self, logits: torch.Tensor) -> torch.Tensor:
         cap = float(self.logit_softcap)
-        return logits if cap <= 0.0 else torch.tanh(logits / cap) * cap
+        return logits if cap <= 0.0 else ops.softcap(logits, cap)
 
     def chunked_output(self, last_hidden_state: torch.Tensor) -> List[torch.Tensor]:
         return [self._cap(self.output(chunk)) for chunk in last_hidden_state.tensor_split(self.num_output_chunks, dim=1)]
@@ -277,13 +311,20 @@ class TransformerDecoder(nn.Module):
         self._validate_inputs(seq_len, mask=mask, encoder_input=encoder_input, encoder_mask=encoder_mask, input_pos=input_pos)
         h = ops.embed_tokens(self.tok_embeddings, tokens) if input_embeds is None else input_embeds
         hidden = []
+        layer_state: dict = {}
+        kinds = [getattr(layer, "inner_cls", type(layer)) for layer in self.layers]
         for i, layer in enumerate(self.layers):
             if i in self.output_hidden_states:
-                hidden.append(h)
-            h = layer(h, mask=mask, encoder_input=encoder_input, encoder_mask=encoder_mask, input_pos=input_pos)
+                hidden.append(h[0] if isinstance(h, tuple) else h)
+            extra = {}
+            if kinds[i] is ResidualStreamLayer:
+                following = getattr(self.layers[i + 1], "sa_norm", None) if i + 1 < len(self.layers) else self.norm
+                extra = {"layer_state": layer_state, "next_norm": following if isinstance(following, StreamRMSNorm) else None}
+            h = layer(h, mask=mask, encoder_input=encoder_input, encoder_mask=encoder_mask, input_pos=input_pos, **extra)
+        h, normed = h if isinstance(h, tuple) else (h, None)
         if len(self.layers) in self.output_hidden_states:
             hidden.append(h)
-        h = self.norm(h)
+        h = self.norm(h) if normed is None else normed
         if self.skip_output_layer:
             output = h
         elif self.num_output_chunks > 0:
@@ -293,6 +334,8 @@ class TransformerDecoder(nn.Module):
         return output if not hidden else [*hidden, output]
 
     def unembed_normed(self, h: torch.Tensor) -> torch.Tensor:
+        if self.wide_logits and type(self.output).__name__ == "Linear" and self.output.bias is None:
+            return self._cap(ops.linear_wide(h, self.output.weight))
         return self._cap(self.output(h).float())
 
     def unembed(self, h: torch.Tensor) -> torch.Tensor:
@@ -300,4 +343,4 @@ class TransformerDecoder(nn.Module):
         h = self.norm(h)
         if self.num_output_chunks > 0:
             return self.chunked_output(h)
-        return self._cap(self.output(h).float())
+        return self.unembed_normed(h)

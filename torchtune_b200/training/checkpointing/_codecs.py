@@ -54,6 +54,7 @@ def _load_family_codecs() -> None:
     import importlib
 
     for mod in (
+        "begapel._convert_weights",
         "phi3._convert_weights",
         "qwen2._convert_weights",
         "qwen3._convert_weights",

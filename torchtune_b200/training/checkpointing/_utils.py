@@ -54,6 +54,7 @@ VAL_DATALOADER_KEY = "val_dataloader"
 class ModelType(Enum):
     """Architecture tag selecting the weight-conversion rules of a checkpointer."""
 
+    BEGAPEL = "begapel"
     GEMMA = "gemma"
     GEMMA2 = "gemma2"
     LLAMA2 = "llama2"
