@@ -25,6 +25,7 @@ from .. import config, training, utils
 from ..config import DictConfig, OmegaConf
 from ..data import Message, load_image, padded_collate, padded_collate_tiled_images_and_mask
 from ..generation import sample
+from ..ops.mask import AttentionMask
 from ..modules.model_fusion import DeepFusionModel, EarlyFusionModel
 
 
@@ -53,8 +54,11 @@ class CachedDecoder:
         self.temperature, self.top_k, self.stop_tokens = temperature, top_k, set(int(t) for t in stop_tokens)
         self._keys = torch.arange(self.total, device=device)
 
-    def visibility(self, first: int, count: int) -> torch.Tensor:
-        """``[1, count, total]`` booleans: the token at position ``first + i`` sees the cache slots ``0 … first + i``."""
+    def visibility(self, first: int, count: int):
+        """``[1, count, total]`` booleans: the token at position ``first + i`` sees the cache slots ``0 … first + i`` (a model that reads
+        its key ranges from the cache position gets just the causal description)."""
+        if getattr(self.forward, "span_masks", False):
+            return AttentionMask(causal=True)
         pos = torch.arange(first, first + count, device=self.device)
         return (self._keys[None, :] <= pos[:, None]).unsqueeze(0)
 

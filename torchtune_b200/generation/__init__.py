@@ -3,7 +3,9 @@ from ._generation import (
     generate_next_token,
     get_causal_mask_from_padding_mask,
     get_position_ids_from_padding_mask,
+    last_logits,
     sample,
 )
+from ._rows import BatchDecoder, RowLayout
 
-__all__ = ["generate", "generate_next_token", "get_causal_mask_from_padding_mask", "get_position_ids_from_padding_mask", "sample"]
+__all__ = ["generate", "generate_next_token", "get_causal_mask_from_padding_mask", "get_position_ids_from_padding_mask", "sample", "last_logits", "BatchDecoder", "RowLayout"]

@@ -6,6 +6,8 @@ from typing import Callable, List, Optional, Tuple
 import torch
 
 from ..modules import TransformerDecoder
+from ..modules.attention import MaskLike
+from ._rows import RowLayout, hidden_states
 
 
 def multinomial_sample_one(probs: torch.Tensor, q: torch.Tensor) -> torch.Tensor:
@@ -39,9 +41,16 @@ def sample(logits: torch.Tensor, *, temperature: float = 1.0, top_k: Optional[in
     return multinomial_sample_one(probs, q)
 
 
+def last_logits(model: TransformerDecoder, x: torch.Tensor, *, input_pos: torch.Tensor, mask: MaskLike) -> torch.Tensor:
+    """Logits ``[b, vocab]`` of the last position; a plain decoder runs its output projection on that position only."""
+    if type(model) is TransformerDecoder and x.shape[1] > 1 and model.num_output_chunks == 0 and not model.output_hidden_states and not model.skip_output_layer:
+        return model.unembed_normed(hidden_states(model, x, input_pos=input_pos, mask=mask)[:, -1:])[:, 0]
+    return model(x, input_pos=input_pos, mask=mask)[:, -1]
+
+
 def generate_next_token(model: TransformerDecoder, input_pos: torch.Tensor, x: torch.Tensor, q: Optional[torch.Tensor] = None, *, mask: Optional[torch.Tensor] = None, temperature: float = 1.0, top_k: Optional[int] = None) -> Tuple[torch.Tensor, torch.Tensor]:
     """One forward pass; samples from the last position.  Returns ``(tokens [b,1], logits [b,1,v])``."""
-    logits = model(x, input_pos=input_pos, mask=mask)[:, -1]
+    logits = last_logits(model, x, input_pos=input_pos, mask=mask)
     return sample(logits.clone(), temperature=temperature, top_k=top_k, q=q), logits.unsqueeze(1)
 
 
@@ -101,7 +110,10 @@ def generate(
     mask_width = model.decoder_max_cache_seq_len if incremental else total_len
 
     real = prompt != pad_id
-    if not real.all():
+    layout = RowLayout(real) if incremental and getattr(model, "span_masks", False) else None
+    if layout is not None:
+        masks = input_pos = None
+    elif not real.all():
         real = torch.nn.functional.pad(real, (0, max_generated_tokens), value=True)
         masks = get_causal_mask_from_padding_mask(real, target_seq_len=mask_width)
         input_pos = get_position_ids_from_padding_mask(real)
@@ -112,8 +124,12 @@ def generate(
     def draw_q():
         return None if rng is None else _exponential_like((bsz, model.tok_embeddings.num_embeddings), device, rng)
 
-    first_mask = masks[:, :prompt_len] if incremental else masks[:, :prompt_len, :prompt_len]
-    tokens, logits = generate_next_token(model, input_pos=input_pos[:, :prompt_len].squeeze(), mask=first_mask, x=prompt, temperature=temperature, top_k=top_k, q=draw_q())
+    if layout is not None:
+        first_mask, first_pos = layout.mask(0, prompt_len), layout.positions(0, prompt_len)
+    else:
+        first_mask = masks[:, :prompt_len] if incremental else masks[:, :prompt_len, :prompt_len]
+        first_pos = input_pos[:, :prompt_len].squeeze()
+    tokens, logits = generate_next_token(model, input_pos=first_pos, mask=first_mask, x=prompt, temperature=temperature, top_k=top_k, q=draw_q())
     out_tokens = torch.cat([prompt, tokens], dim=-1)
     logit_steps = [logits] if return_logits else None  # joined once at the end: joining every step copies the whole history each time
     pos = prompt_len
@@ -137,7 +153,9 @@ def generate(
     for _ in range(max_generated_tokens - 1):
         if stop is not None:
             keep = torch.cat([keep, (~reached).reshape(bsz, 1).to(torch.int32)], dim=-1)
-        if incremental:
+        if layout is not None:
+            cur_pos, cur_mask, x = layout.positions(pos, 1), layout.mask(pos, 1), tokens.clone()
+        elif incremental:
             cur_pos, cur_mask, x = input_pos[:, pos].contiguous(), masks[:, pos, None, :].contiguous(), tokens.clone()
         else:
             cur_pos, cur_mask, x = input_pos[:, : pos + 1], masks[:, : pos + 1, : pos + 1], out_tokens.clone()

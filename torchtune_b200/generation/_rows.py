@@ -1,0 +1,129 @@
+"""Batches of rows that start together and go on one token at a time.
+
+Prompts of unequal length are padded on the left, so all rows append at the same cache slot.  :class:`RowLayout` knows where each row
+begins and gives the positions and the visible keys of any range of slots; :class:`BatchDecoder` runs a model on its KV caches with it,
+returning hidden states, and gives up rows that are finished."""
+from __future__ import annotations
+
+from typing import List, Optional, Sequence
+
+import torch
+
+from ..modules import TransformerDecoder
+from ..modules.attention import MaskLike
+from ..modules.common_utils import delete_kv_caches
+from ..ops.mask import AttentionMask
+
+
+def hidden_states(model: TransformerDecoder, x: torch.Tensor, *, input_pos: torch.Tensor, mask: MaskLike) -> torch.Tensor:
+    """Normalised hidden states ``[b, s, d]`` in front of the output projection."""
+    before = model.skip_output_layer
+    model.skip_output_layer = True
+    try:
+        return model(x, input_pos=input_pos, mask=mask)
+    finally:
+        model.skip_output_layer = before
+
+
+class RowLayout:
+    """Cache slots of left-padded rows: ``real`` ``[b, s]`` is True on prompt tokens, every later slot is a real token of its row."""
+
+    def __init__(self, real: torch.Tensor) -> None:
+        n = real.shape[1]
+        padded = not bool(real.all())
+        slots = torch.arange(n, device=real.device)
+        if padded and not bool((real == (slots[None, :] >= n - real.sum(1, keepdim=True))).all()):
+            # a pad id inside a prompt: the row starts at its first real token and what follows counts as tokens
+            first = torch.where(real.any(1), real.to(torch.int8).argmax(1), n)
+        else:
+            first = n - real.sum(1)
+        self.start = first.to(torch.int32)
+        self.padded = padded
+        self.batch = real.shape[0]
+
+    def positions(self, first: int, count: int) -> torch.Tensor:
+        """``[b, count]`` int32 positions of the slots ``first …``, counted from each row's own first token (0 on padding)."""
+        slots = torch.arange(first, first + count, dtype=torch.int32, device=self.start.device)
+        return (slots[None, :] - self.start[:, None]).clamp_min_(0)
+
+    def mask(self, first: int, count: int) -> AttentionMask:
+        return AttentionMask(causal=True, key_start=self.start, query_start=first)
+
+    def keep(self, rows: Sequence[int]) -> None:
+        self.start = self.start[list(rows)].contiguous()
+        self.batch = len(rows)
+
+
+class BatchDecoder:
+    """One batch at a time on a model's KV caches: :meth:`begin`, then :meth:`advance` until every row has been ended.
+
+    ``max_tokens`` is the most tokens that live rows hold together; the caches of a batch are sized from it (padding included)."""
+
+    def __init__(self, model: TransformerDecoder, device: torch.device, dtype: torch.dtype, max_tokens: int) -> None:
+        if not getattr(model, "span_masks", False):
+            raise ValueError("this decoder needs a model that takes its key ranges from row starts")
+        self.model, self.device, self.dtype, self.max_tokens = model, device, dtype, int(max_tokens)
+        self.layout: Optional[RowLayout] = None
+        self.used = 0
+        self._capacity = (0, 0)
+
+    @property
+    def rows(self) -> int:
+        return 0 if self.layout is None else self.layout.batch
+
+    def _reserve(self, batch: int, slots: int) -> None:
+        if batch > self._capacity[0] or slots > self._capacity[1]:
+            if self.model.caches_are_setup():
+                delete_kv_caches(self.model)
+            with self.device:
+                self.model.setup_caches(batch, self.dtype, decoder_max_seq_len=slots)
+            self._capacity = (batch, slots)
+        else:
+            self.model.reset_caches()
+
+    def begin(self, prompts: List[List[int]]) -> torch.Tensor:
+        """Hidden states ``[b, longest, d]`` of new rows; row ``i`` occupies the last ``len(prompts[i])`` places."""
+        if self.rows:
+            raise RuntimeError("the batch before has unfinished rows")
+        lengths = [len(p) for p in prompts]
+        longest, shortest = max(lengths), min(lengths)
+        if shortest < 1:
+            raise ValueError("a row starts with at least one token")
+        # a row may go on alone until it holds every token of the budget: that many slots behind the padding of the shortest one
+        self._reserve(len(prompts), longest + max(self.max_tokens - shortest, 0))
+        tokens = torch.tensor([[0] * (longest - n) + p for p, n in zip(prompts, lengths)], device=self.device)
+        real = torch.arange(longest)[None, :] >= torch.tensor([longest - n for n in lengths])[:, None]
+        self.layout, self.used = RowLayout(real.to(self.device)), 0
+        return self._run(tokens)
+
+    def advance(self, tokens: List[int]) -> torch.Tensor:
+        """Hidden states ``[b, 1, d]`` of one more token per live row."""
+        if len(tokens) != self.rows or not tokens:
+            raise ValueError(f"{len(tokens)} tokens for {self.rows} rows")
+        return self._run(torch.tensor(tokens, device=self.device)[:, None])
+
+    def _run(self, tokens: torch.Tensor) -> torch.Tensor:
+        first, count = self.used, tokens.shape[1]
+        h = hidden_states(self.model, tokens, input_pos=self.layout.positions(first, count), mask=self.layout.mask(first, count))
+        self.used += count
+        return h
+
+    def logits(self, hidden: torch.Tensor) -> torch.Tensor:
+        """fp32 logits of hidden states ``[..., d]``."""
+        return self.model.unembed_normed(hidden)
+
+    def end(self, rows: Sequence[int]) -> None:
+        """Gives up rows (indices into the live ones); the others close ranks, so later :meth:`advance` calls name only them."""
+        gone = set(rows)
+        kept = [i for i in range(self.rows) if i not in gone]
+        if not kept:
+            self.layout, self.used = None, 0
+            self.model.reset_caches()
+            return
+        if len(kept) == self.rows:
+            return
+        for layer in self.model.layers:
+            cache = layer.attn.kv_cache
+            if cache is not None:
+                cache.keep_rows(kept)
+        self.layout.keep(kept)
