@@ -587,6 +587,111 @@ def run_ours_sharded(args) -> dict:
     return out if rank == 0 else {}
 
 
+# Serving comparison (``--serve``): a Begapel decoder and the closest other decoder of equal width, heads, feed-forward and depth.
+SERVE_SIZES = {
+    "1b": dict(width=2048, heads=16, ff=8192, layers=12, vocab=65_536),
+    "3b": dict(width=4096, heads=32, ff=14_336, layers=8, vocab=65_536),
+}
+SERVE_ROT, SERVE_RANK, SERVE_DIM = 64, 512, 128
+
+
+def run_serve(args) -> dict:
+    """Prefill and decode throughput through the generation path, random weights: ``--serve 1b | 3b``.  Begapel layers (every fourth one
+    without latents of its own) against llama3_1 layers with a quarter as many key heads."""
+    import torch
+
+    from torchtune_b200 import training
+    from torchtune_b200.generation import DecodeGraph, RowLayout, generate_next_token
+    from torchtune_b200.models._registry import build_from_config
+    from torchtune_b200.models.llama3_1 import llama3_1
+    from torchtune_b200.modules import delete_kv_caches
+    from torchtune_b200.ops._lib import check_device_errors, lib
+
+    z = SERVE_SIZES[args.serve]
+    dev, prompt, context = torch.device("cuda", 0), 8192, 4096
+    torch.manual_seed(0)
+
+    def mixer(i):
+        m = {"heads": z["heads"], "dim": SERVE_DIM, "rot_dim": SERVE_ROT, "vdim": SERVE_DIM, "kv_rank": SERVE_RANK, "rot": {"base": 10000.0, "dims": SERVE_ROT}, "scale": (SERVE_DIM + SERVE_ROT) ** -0.5}
+        return {**m, "kv_from": i - 1} if i % 4 == 3 else m
+
+    cfg = {"architecture": "Begapel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 30.0,
+           "layers": [{"type": "latent_attention", "mixer": mixer(i), "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(z["layers"])]}
+    builders = {
+        "begapel": lambda: build_from_config(cfg, max_seq_len=16384),
+        "llama3_1": lambda: llama3_1(vocab_size=z["vocab"], num_layers=z["layers"], num_heads=z["heads"], num_kv_heads=z["heads"] // 4, embed_dim=z["width"], max_seq_len=16384,
+                                     intermediate_dim=z["ff"]),
+    }
+
+    def timed(fn, n):
+        for i in range(max(3, args.warmup)):
+            fn(i)
+        torch.cuda.synchronize()
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        for i in range(n):
+            fn(i)
+        e1.record()
+        torch.cuda.synchronize()
+        return e0.elapsed_time(e1) / n
+
+    results, sampler = {}, ClockSampler(0)
+    torch.cuda.synchronize()
+    sampler.start()
+    launches0 = lib().ttb_launch_count()
+    with torch.inference_mode():
+        for name, build in builders.items():
+            with training.set_default_dtype(torch.bfloat16), dev:
+                model = build().eval()
+            for p in model.parameters():
+                if p.dim() == 2:
+                    p.normal_(0, p.shape[1] ** -0.5)
+            res = {"params_m": round(sum(p.numel() for p in model.parameters()) / 1e6)}
+            spans = model.span_masks
+            for b in (1, 4):
+                s = prompt // b
+                with dev:
+                    model.setup_caches(b, torch.bfloat16, decoder_max_seq_len=s)
+                x = torch.randint(0, z["vocab"], (b, s), device=dev)
+                layout = RowLayout(torch.ones(b, s, dtype=torch.bool, device=dev))
+                mask = layout.mask(0, s) if spans else torch.tril(torch.ones(s, s, dtype=torch.bool, device=dev)).unsqueeze(0)
+                pos = layout.positions(0, s) if spans else torch.arange(s, device=dev).unsqueeze(0)
+
+                def prefill(_):
+                    model.reset_caches()
+                    generate_next_token(model, input_pos=pos, x=x, mask=mask)
+
+                res[f"prefill_b{b}_tokens_per_s"] = round(b * s / timed(prefill, args.steps) * 1e3)
+                delete_kv_caches(model)
+            for b in (1, 16, 64):
+                width = context + 256
+                with dev:
+                    model.setup_caches(b, torch.bfloat16, decoder_max_seq_len=width)
+                x = torch.randint(0, z["vocab"], (b, 1), device=dev)
+                layout = RowLayout(torch.ones(b, context, dtype=torch.bool, device=dev))
+                for layer in model.layers:  # a context of zeros: timing does not depend on the values
+                    cache = layer.attn.kv_cache
+                    if cache is not None:
+                        cache.advance(context) if spans else cache.cache_pos.add_(context)
+                if spans:
+                    graph = DecodeGraph(model, layout)
+                    step = lambda i: model.unembed_normed(graph(x))  # noqa: E731
+                else:
+                    masks = torch.tril(torch.ones(width, width, dtype=torch.bool, device=dev)).unsqueeze(0)
+                    step = lambda i: generate_next_token(model, input_pos=torch.full((b, 1), context + i, device=dev), x=x, mask=masks[:, context + i, None, :].contiguous())  # noqa: E731
+                res[f"decode_b{b}_tokens_per_s"] = round(b / timed(step, max(10, args.steps)) * 1e3)
+                delete_kv_caches(model)
+            results[name] = res
+            del model
+            torch.cuda.empty_cache()
+    clocks = sampler.stop()
+    check_device_errors()
+    return {"metric": "serving_tokens_per_second", "value": results["begapel"]["decode_b16_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+            "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic tokens, random-init weights", "impl": "ours",
+            "config": {"serve": args.serve, **z, "prompt_tokens": prompt, "decode_context": context, "l2": "weights and caches larger than L2"}, "results": results, "clocks": clocks,
+            "gpu_launches": int(lib().ttb_launch_count() - launches0)}
+
+
 def run_reference(args) -> dict:
     from baseline.reference_arm import run as run_ref
     from baseline.reference_arm import run_peft
@@ -616,13 +721,16 @@ def main() -> None:
     ap.add_argument("--ref-compile", action="store_true", help="with --impl reference: the reference's `compile: True` path (informational; the default arm stays on the stock eager path)")
     ap.add_argument("--fp8-recipe", choices=["tensorwise", "blockwise"], default="tensorwise", help="with --fp8: one scale per tensor, or MX block scales (32 values per scale)")
     ap.add_argument("--fp8", action="store_true", help="variant: fp8 decoder linears (the headline number is always bf16)")
+    ap.add_argument("--serve", choices=sorted(SERVE_SIZES), default=None, help="prefill and decode throughput of Begapel layers beside llama3_1 layers of equal size, instead of the training step")
     args = ap.parse_args()
     rank, world, _ = dist_env()
     if args.gpus > 1 and world == 1:
         # convenience: re-launch under torchrun when called directly with --gpus N
         cmd = [sys.executable, "-m", "torch.distributed.run", "--nnodes=1", f"--nproc-per-node={args.gpus}", "--master-addr", "127.0.0.1", "--master-port", "29511", __file__, *sys.argv[1:]]
         sys.exit(subprocess.call(cmd))
-    if args.impl == "reference":
+    if args.serve:
+        result = {"impl": "reference", "unavailable": "--serve compares models of this package"} if args.impl == "reference" else run_serve(args)
+    elif args.impl == "reference":
         result = run_reference(args)
     else:
         if args.config != "8b":

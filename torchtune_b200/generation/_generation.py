@@ -7,7 +7,7 @@ import torch
 
 from ..modules import TransformerDecoder
 from ..modules.attention import MaskLike
-from ._rows import RowLayout, hidden_states
+from ._rows import DecodeGraph, RowLayout, hidden_states
 
 
 def multinomial_sample_one(probs: torch.Tensor, q: torch.Tensor) -> torch.Tensor:
@@ -150,6 +150,13 @@ def generate(
             return out_tokens, (logits if return_logits else None)
 
     step_fn = custom_generate_next_token or generate_next_token
+    if layout is not None and custom_generate_next_token is None and device.type == "cuda" and max_generated_tokens > 2:
+        graph = DecodeGraph(model, layout)
+
+        def step_fn(model, input_pos, x, q=None, *, mask=None, temperature=1.0, top_k=None):
+            logits = model.unembed_normed(graph(x))[:, -1]
+            return sample(logits, temperature=temperature, top_k=top_k, q=q), logits.unsqueeze(1)
+
     for _ in range(max_generated_tokens - 1):
         if stop is not None:
             keep = torch.cat([keep, (~reached).reshape(bsz, 1).to(torch.int32)], dim=-1)

@@ -54,18 +54,70 @@ class RowLayout:
         self.batch = len(rows)
 
 
+class DecodeGraph:
+    """The one-token step of a batch as a CUDA graph: embedding to final norm with every launch recorded once, the cache slot held on the
+    device and moved on by the graph itself.  Calling it with ``[b, 1]`` tokens replays the step on the model's caches; the result lives
+    in a buffer that the next call overwrites."""
+
+    def __init__(self, model: TransformerDecoder, layout: RowLayout) -> None:
+        self.caches = [layer.attn.kv_cache for layer in model.layers if layer.attn.kv_cache is not None]
+        used = self.caches[0].size
+        dev = layout.start.device
+        self.batch = layout.batch
+        self.tokens = torch.zeros(self.batch, 1, dtype=torch.int64, device=dev)
+        self.start = layout.start
+        self.slot = torch.tensor([used], dtype=torch.int32, device=dev)
+        mask = layout.mask(used, 1)
+
+        def body() -> torch.Tensor:
+            for c in self.caches:
+                c.rewind(used)
+            return hidden_states(model, self.tokens, input_pos=(self.slot - self.start).clamp_min_(0)[:, None], mask=mask)
+
+        for c in self.caches:
+            c.slot = self.slot
+        try:
+            side = torch.cuda.Stream(device=dev)
+            side.wait_stream(torch.cuda.current_stream(dev))
+            with torch.cuda.stream(side):  # first launches and their one-time set-up stay out of the recording
+                body()
+            torch.cuda.current_stream(dev).wait_stream(side)
+            self.graph = torch.cuda.CUDAGraph()
+            with torch.cuda.graph(self.graph):
+                self.hidden = body()
+                self.slot.add_(1)
+        finally:
+            for c in self.caches:
+                c.slot = None
+                c.rewind(used)
+        self._next = used
+
+    def __call__(self, tokens: torch.Tensor) -> torch.Tensor:
+        at = self.caches[0].reserve(self.batch, 1)
+        if at != self._next:
+            self.slot.fill_(at)
+        self.tokens.copy_(tokens.view(self.batch, 1))
+        self.graph.replay()
+        for c in self.caches:
+            c.advance(1)
+        self._next = at + 1
+        return self.hidden
+
+
 class BatchDecoder:
     """One batch at a time on a model's KV caches: :meth:`begin`, then :meth:`advance` until every row has been ended.
 
     ``max_tokens`` is the most tokens that live rows hold together; the caches of a batch are sized from it (padding included)."""
 
-    def __init__(self, model: TransformerDecoder, device: torch.device, dtype: torch.dtype, max_tokens: int) -> None:
+    def __init__(self, model: TransformerDecoder, device: torch.device, dtype: torch.dtype, max_tokens: int, graphs: bool = True) -> None:
         if not getattr(model, "span_masks", False):
             raise ValueError("this decoder needs a model that takes its key ranges from row starts")
         self.model, self.device, self.dtype, self.max_tokens = model, device, dtype, int(max_tokens)
         self.layout: Optional[RowLayout] = None
         self.used = 0
         self._capacity = (0, 0)
+        self._graphs = graphs and device.type == "cuda"
+        self._graph: Optional[DecodeGraph] = None
 
     @property
     def rows(self) -> int:
@@ -100,7 +152,13 @@ class BatchDecoder:
         """Hidden states ``[b, 1, d]`` of one more token per live row."""
         if len(tokens) != self.rows or not tokens:
             raise ValueError(f"{len(tokens)} tokens for {self.rows} rows")
-        return self._run(torch.tensor(tokens, device=self.device)[:, None])
+        step = torch.tensor(tokens, device=self.device)[:, None]
+        if not self._graphs:
+            return self._run(step)
+        if self._graph is None:
+            self._graph = DecodeGraph(self.model, self.layout)
+        self.used += 1
+        return self._graph(step).clone()
 
     def _run(self, tokens: torch.Tensor) -> torch.Tensor:
         first, count = self.used, tokens.shape[1]
@@ -117,11 +175,12 @@ class BatchDecoder:
         gone = set(rows)
         kept = [i for i in range(self.rows) if i not in gone]
         if not kept:
-            self.layout, self.used = None, 0
+            self.layout, self.used, self._graph = None, 0, None
             self.model.reset_caches()
             return
         if len(kept) == self.rows:
             return
+        self._graph = None
         for layer in self.model.layers:
             cache = layer.attn.kv_cache
             if cache is not None:

@@ -72,6 +72,12 @@ class LatentCache(nn.Module):
     def advance(self, count: int) -> None:
         self._size += count
 
+    def rewind(self, size: int) -> None:
+        """Forgets the tokens from slot ``size`` on."""
+        if not 0 <= size <= self.max_seq_len:
+            raise ValueError(f"{size} is outside the cache")
+        self._size = size
+
     def keep_rows(self, rows: List[int]) -> None:
         """Drops every batch row that is not in ``rows`` (increasing) and moves the kept ones to the front."""
         for to, row in enumerate(rows):

@@ -108,12 +108,13 @@ def _declare(L: ctypes.CDLL) -> None:
     L.ttb_latent_decode.argtypes = [vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, i32, vp, i64, vp, i64, f32, vp, vp]
     L.ttb_latent_prepare.argtypes = [vp, i64, vp, vp, i64, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32, f32, i32, vp]
     L.ttb_latent_absorb.argtypes = [vp, i64, i32, vp, vp, i64, i32, i32, i32, i32, i32, i32, vp]
-    L.ttb_latent_value.argtypes = [vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, i32, vp]
-    L.ttb_latent_combine.argtypes = [vp, vp, vp, i32, i32, i32, i32, vp]
+    L.ttb_latent_value.argtypes = [vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, vp]
+    L.ttb_latent_combine.argtypes = [vp, vp, vp, i32, i32, i32, i32, i32, vp]
     L.ttb_latent_gate_rows.argtypes = [vp, vp, i64, vp, i32, i32, i32, vp]
     L.ttb_latent_attention_any.argtypes = [vp, i64, i64, i64, vp, i64, i64, i64, vp, i64, i64, vp, i64, i64, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32,
                                            vp, i32, vp, i64, i64, vp, i64, i64, f32, i32, vp]
-    for fn in (L.ttb_residual_norm, L.ttb_softcap, L.ttb_latent_prefill, L.ttb_latent_decode, L.ttb_latent_prepare, L.ttb_latent_absorb, L.ttb_latent_value, L.ttb_latent_combine,
+    L.ttb_latent_decode_tile.argtypes = [i32, i32, i32]
+    for fn in (L.ttb_residual_norm, L.ttb_softcap, L.ttb_latent_decode_tile, L.ttb_latent_prefill, L.ttb_latent_decode, L.ttb_latent_prepare, L.ttb_latent_absorb, L.ttb_latent_value, L.ttb_latent_combine,
                L.ttb_latent_gate_rows, L.ttb_latent_attention_any):
         fn.restype = i32
     for fn in (L.ttb_moe_route_sort, L.ttb_moe_permute_indices, L.ttb_embedding_fwd, L.ttb_embedding_bwd):

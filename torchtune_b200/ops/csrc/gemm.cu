@@ -859,6 +859,10 @@ static int launch_gemm(const void* A, const void* B, const GemmParams& p, long l
 template <bool A_MN, bool B_MN>
 static int dispatch_bn(const void* A, const void* B, const GemmParams& p, long long lda, long long ldb,
                        cudaStream_t stream, const SecondPair& sp = SecondPair()) {
+  // One row of tiles (decoding) streams the weights: narrower tiles put more SMs to work.
+  const bool one_row = p.M <= BM && p.splits == 1;
+  if (one_row && p.N > 64 && (p.N + 127) / 128 <= sm_count() / 2) return launch_gemm<64, A_MN, B_MN>(A, B, p, lda, ldb, stream, sp);
+  if (one_row && p.N > 128 && (p.N + 255) / 256 <= sm_count() / 2) return launch_gemm<128, A_MN, B_MN>(A, B, p, lda, ldb, stream, sp);
   if (p.N > 128) return launch_gemm<256, A_MN, B_MN>(A, B, p, lda, ldb, stream, sp);
   if (p.N > 64) return launch_gemm<128, A_MN, B_MN>(A, B, p, lda, ldb, stream, sp);
   return launch_gemm<64, A_MN, B_MN>(A, B, p, lda, ldb, stream, sp);

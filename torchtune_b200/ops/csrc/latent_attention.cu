@@ -12,7 +12,7 @@
 //   outputs in tensor memory (the scheme of attention_fwd2.cu); the epilogue multiplies by the sigmoid of a gate row.
 //
 // * decode (`latent_decode_kernel`): one query per sequence, queries already multiplied by W_ukᵀ.  All heads share the keys, so a
-//   tile of 128 cached rows is loaded once and used twice: Sᵀ = C · Qᵀ (M = 128 keys, N = heads) and Oᵀ += Cᵀ · Pᵀ (M = 128 latent
+//   tile of cached rows is loaded once and used twice: Sᵀ = C · Qᵀ (M = keys, N = heads) and Oᵀ += Cᵀ · Pᵀ (M = 128 latent
 //   columns, N = heads).  Heads sit in the N dimension, so 16 heads cost 16 columns rather than a padded 128-row tile.  Cache
 //   rows are cut over CTAs (split keys); the partial outputs are combined by the value projection.
 //
@@ -28,6 +28,14 @@ namespace latent {
 using namespace attn;
 
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + __expf(-z)); }
+
+// Up to four contraction steps (of 16 columns) of one pair of 64-column K-major panels.  `da` / `db` describe the panels' first steps; a step
+// further is 32 bytes, i.e. 2 in the descriptors' address fields, so the issuing thread spends one addition per operand.
+__device__ __forceinline__ void umma_panel(uint32_t d, uint64_t da, uint64_t db, int steps, uint32_t idesc, bool accumulate) {
+#pragma unroll
+  for (int k = 0; k < 4; ++k)
+    if (k < steps) umma_f16(d, da + 2 * k, db + 2 * k, idesc, accumulate || k > 0);
+}
 
 // ===================================================================================== prefill
 struct PrefillParams {
@@ -181,10 +189,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       }
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t q_base = aQ + x * q_bytes, k_base = aK + st * q_bytes;
-        for (int k = 0; k < p.dim_steps; ++k) umma_f16(tS[x], desc_kmajor(q_base, k), desc_kmajor(k_base, k), idesc_s, k != 0);
-        const uint32_t off = p.dim_panels * kPanelBytes;
-        for (int k = 0; k < p.rot_steps; ++k) umma_f16(tS[x], desc_kmajor(q_base + off, k), desc_kmajor(k_base + off, k), idesc_s, 1);
+        uint64_t dq = desc_kmajor(aQ + x * q_bytes, 0), dk = desc_kmajor(aK + st * q_bytes, 0);
+        for (int c = 0; c < p.dim_panels; ++c, dq += kPanelBytes >> 4, dk += kPanelBytes >> 4) umma_panel(tS[x], dq, dk, p.dim_steps - 4 * c, idesc_s, c > 0);
+        for (int c = 0; c < p.rot_panels; ++c, dq += kPanelBytes >> 4, dk += kPanelBytes >> 4) umma_panel(tS[x], dq, dk, p.rot_steps - 4 * c, idesc_s, true);
         umma_commit(&s_full[x]);
         const bool other_later = (x == 0) && active(1, j);  // tile 1 issues its S(j) after tile 0's
         if (!other_later) umma_commit(&k_empty[st]);
@@ -212,9 +219,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         }
         tc_fence_after();
         if (lane == 0) {
-          const uint32_t v_base = aV + st * v_bytes;
+          const uint64_t dv = desc_mnmajor(aV + st * v_bytes, 0);
 #pragma unroll
-          for (int k = 0; k < kBlk / 16; ++k) umma_f16_ts(tO[x], tS[x] + k * 8, desc_mnmajor(v_base, k), idesc_o, (n | k) != 0);
+          for (int k = 0; k < kBlk / 16; ++k) umma_f16_ts(tO[x], tS[x] + k * 8, dv + k * (2048 >> 4), idesc_o, (n | k) != 0);
           const bool other_later = (x == 0) && active(1, j);
           if (!other_later) umma_commit(&v_empty[st]);
           if (n + 1 == count[x]) umma_commit(&o_done[x]);
@@ -409,8 +416,7 @@ struct DecodeParams {
 };
 
 static constexpr int kDecodeThreads = 256;
-static constexpr int kPairBytes = 2 * kPanelBytes;
-static constexpr int kMaxRing = 8;
+static constexpr int kMaxRing = 12;
 static constexpr int kDecodeBarriers = 2 * kMaxRing + 4 + 4 + 3;
 
 __device__ __forceinline__ float warp_max(float v) {
@@ -444,18 +450,21 @@ __device__ __forceinline__ void tmem_st_heads(uint32_t addr, const uint32_t (&v)
   else tmem_st_32x32(addr, v);
 }
 
-// HN: heads per CTA (16 or 32)
-template <int HN>
+// HN: heads per CTA (16 or 32).  KB: keys per tile.  A wide latent leaves room for one and a bit 128-key tiles; tiles of 64 keys are then
+// double-buffered instead.  Their score MMA still has 128 rows: the upper 64 read whatever follows the panel in shared memory (always
+// inside the allocation) and are never looked at.
+template <int HN, int KB>
 __global__ void __launch_bounds__(kDecodeThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmR, DecodeParams p) {
   constexpr int kQPanel = HN * 128;  // bytes of a 64-column panel of HN rows
+  constexpr int kKeyPanel = KB * 128, kPairBytes = 2 * kKeyPanel;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* sC = smem;                                        // [ring] pieces: 128 rows x 128 columns
+  uint8_t* sC = smem;                                        // [ring] pieces: KB rows x 128 columns
   uint8_t* sR = sC + p.ring * kPairBytes;                    // [rot_stages]
-  uint8_t* sQ = sR + p.rot_stages * p.rot_panels * kPanelBytes;  // 2 * pairs latent panels, then the rotated ones
-  uint8_t* sP = sQ + (2 * p.pairs + p.rot_panels) * kQPanel;     // [HN heads, 128 keys]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kQPanel);
+  uint8_t* sQ = sR + p.rot_stages * p.rot_panels * kKeyPanel;  // 2 * pairs latent panels, then the rotated ones
+  uint8_t* sP = sQ + (2 * p.pairs + p.rot_panels) * kQPanel;     // [HN heads, KB keys]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + KB / 64 * kQPanel);
   uint64_t* c_full = bars;                 // [ring]
   uint64_t* c_empty = bars + kMaxRing;     // [ring]
   uint64_t* r_full = bars + 2 * kMaxRing;  // [rot_stages <= 2]
@@ -474,8 +483,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int newest = p.slot != nullptr ? *p.slot : p.slot_host;
   const int hi = min(p.hi != nullptr ? p.hi[bi * p.hi_row] : newest, p.slots - 1);
   const int lo = max(p.lo != nullptr ? p.lo[bi * p.lo_row] : 0, 0);
-  const int blk0 = lo / kBlk;
-  const int total = hi >= lo ? hi / kBlk - blk0 + 1 : 0;
+  const int blk0 = lo / KB;
+  const int total = hi >= lo ? hi / KB - blk0 + 1 : 0;
   const int per = (total + splits - 1) / splits;
   const int first = blk0 + split * per;
   const int n_blocks = max(min(per, total - split * per), 0);
@@ -518,14 +527,14 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     int cs = 0, rs = 0;
     uint32_t cph = 0, rph = 0;
     for (int it = 0; it < n_blocks && !*abort_flag; ++it) {
-      const int key0 = (first + it) * kBlk;
+      const int key0 = (first + it) * KB;
       bool ok = true;
       for (int u = 0; u < p.pairs && ok; ++u) {
         ok = mbar_wait(&c_empty[cs], cph ^ 1);
         if (ok && lane == 0) {
           mbar_arrive_expect_tx(&c_full[cs], kPairBytes);
           tma_load_3d(sC + cs * kPairBytes, &tmC, &c_full[cs], u * 128, key0, bi);
-          tma_load_3d(sC + cs * kPairBytes + kPanelBytes, &tmC, &c_full[cs], u * 128 + 64, key0, bi);
+          tma_load_3d(sC + cs * kPairBytes + kKeyPanel, &tmC, &c_full[cs], u * 128 + 64, key0, bi);
         }
         __syncwarp();
         if (++cs == p.ring) cs = 0, cph ^= 1;
@@ -536,9 +545,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         break;
       }
       if (lane == 0) {
-        uint8_t* dst = sR + rs * p.rot_panels * kPanelBytes;
-        mbar_arrive_expect_tx(&r_full[rs], p.rot_panels * kPanelBytes);
-        for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(dst + j * kPanelBytes, &tmR, &r_full[rs], j * 64, key0, bi);
+        uint8_t* dst = sR + rs * p.rot_panels * kKeyPanel;
+        mbar_arrive_expect_tx(&r_full[rs], p.rot_panels * kKeyPanel);
+        for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(dst + j * kKeyPanel, &tmR, &r_full[rs], j * 64, key0, bi);
       }
       __syncwarp();
       if (++rs == p.rot_stages) rs = 0, rph ^= 1;
@@ -548,27 +557,28 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     constexpr uint32_t idesc_s = make_idesc_bf16(128, HN, false, false);
     constexpr uint32_t idesc_o = make_idesc_bf16(128, HN, true, false);
     const uint32_t aC = smem_u32(sC), aR = smem_u32(sR), aQ = smem_u32(sQ), aP = smem_u32(sP);
-    auto q_desc = [&](int panel, int k) { return make_smem_desc_sw128(aQ + panel * kQPanel + (k & 3) * 32, 16, 1024); };
+    const uint64_t dC = make_smem_desc_sw128(aC, 16, 1024), dR = make_smem_desc_sw128(aR, 16, 1024), dQ = make_smem_desc_sw128(aQ, 16, 1024);
+    const uint64_t dCt = make_smem_desc_sw128(aC, kKeyPanel, 1024), dP = make_smem_desc_sw128(aP, 16, 1024);
     auto issue_s = [&](int it) -> bool {
       const int st = it & 1, rs = it % p.rot_stages;
       if (!mbar_wait(&s_free[st], ((it >> 1) & 1) ^ 1)) return false;
-      int step = 0;
       for (int u = 0; u < p.pairs; ++u) {
         const int n = it * p.pairs + u, slot = n % p.ring;
         if (!mbar_wait(&c_full[slot], (n / p.ring) & 1)) return false;
         tc_fence_after();
-        const int stop = min(step + 8, p.c_steps);
-        if (lane == 0)
-          for (int k = step; k < stop; ++k)
-            umma_f16(tS[st], desc_kmajor(aC + slot * kPairBytes, k - step), q_desc(k >> 2, k), idesc_s, k != 0);
+        if (lane == 0) {
+          const uint64_t da = dC + slot * (kPairBytes >> 4), db = dQ + u * (2 * kQPanel >> 4);
+          const int steps = p.c_steps - 8 * u;
+          umma_panel(tS[st], da, db, steps, idesc_s, u > 0);
+          umma_panel(tS[st], da + (kKeyPanel >> 4), db + (kQPanel >> 4), steps - 4, idesc_s, true);
+        }
         __syncwarp();
-        step = stop;
       }
       if (!mbar_wait(&r_full[rs], (it / p.rot_stages) & 1)) return false;
       tc_fence_after();
       if (lane == 0) {
-        const uint32_t base = aR + rs * p.rot_panels * kPanelBytes;
-        for (int k = 0; k < p.rot_steps; ++k) umma_f16(tS[st], desc_kmajor(base, k), q_desc(2 * p.pairs + (k >> 2), k), idesc_s, 1);
+        for (int j = 0; j < p.rot_panels; ++j)
+          umma_panel(tS[st], dR + (rs * p.rot_panels + j) * (kKeyPanel >> 4), dQ + (2 * p.pairs + j) * (kQPanel >> 4), p.rot_steps - 4 * j, idesc_s, true);
         umma_commit(&r_empty[rs]);
         umma_commit(&s_full[st]);
       }
@@ -587,10 +597,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       if (lane == 0) {
         for (int u = 0; u < p.pairs; ++u) {
           const int slot = (it * p.pairs + u) % p.ring;
+          const uint64_t da = dCt + slot * (kPairBytes >> 4);
 #pragma unroll
-          for (int k = 0; k < kBlk / 16; ++k)
-            umma_f16(tO + u * HN, desc_mnmajor(aC + slot * kPairBytes, k), make_smem_desc_sw128(aP + (k >> 2) * kQPanel + (k & 3) * 32, 16, 1024), idesc_o,
-                     (it | k) != 0);
+          for (int k = 0; k < KB / 16; ++k)
+            umma_f16(tO + u * HN, da + k * (2048 >> 4), dP + (k >> 2) * (kQPanel >> 4) + (k & 3) * 2, idesc_o, (it | k) != 0);
           umma_commit(&c_empty[slot]);
         }
         umma_commit(pv_done);
@@ -612,7 +622,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     bool ok = true;
     for (int it = 0; it < n_blocks; ++it) {
       const int st = it & 1;
-      const int key = (first + it) * kBlk + r;
+      const int key = (first + it) * KB + r;
       if (ok && !*abort_flag) ok = mbar_wait(&s_full[st], (it >> 1) & 1);
       tc_fence_after();
       uint32_t sv[HN];
@@ -621,7 +631,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[st]);
-      const bool visible = key >= lo && key <= hi;
+      const bool visible = r < KB && key >= lo && key <= hi;
       bool grows = false;
 #pragma unroll
       for (int h = 0; h < HN; ++h) {
@@ -669,7 +679,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           tmem_st_wait();
         }
       }
-      {
+      if (r < KB) {
         uint8_t* panel = sP + (r >> 6) * kQPanel;
         const int chunk = (r & 63) >> 3, byte = (r & 7) * 2;
 #pragma unroll
@@ -726,18 +736,31 @@ static int map3(CUtensorMap* m, const void* base, uint64_t d0, uint64_t d1, uint
   return make_tmap_3d(m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, d0, d1, d2, s1_elems * 2, s2_elems * 2, 64, b1, b2, CU_TENSOR_MAP_SWIZZLE_128B);
 }
 
-template <int HN>
-static int launch_decode(DecodeParams& p, const void* q, const void* cache, int splits, cudaStream_t st) {
-  const int q_panel = HN * 128;
-  const int fixed = (2 * p.pairs + p.rot_panels) * q_panel + 2 * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
-  const int rot_bytes = p.rot_panels * kPanelBytes;
-  p.rot_stages = fixed + 2 * rot_bytes + 2 * p.pairs * kPairBytes <= kSmemLimit ? 2 : 1;
-  int ring = (kSmemLimit - fixed - p.rot_stages * rot_bytes) / kPairBytes;
-  if (ring > 2 * p.pairs + 1) ring = 2 * p.pairs + 1;
+// Shared memory of one CTA: fixed part and how many 128-column pieces fit next to it.
+template <int HN, int KB>
+static int plan_decode(DecodeParams& p) {
+  const int q_panel = HN * 128, key_panel = KB * 128;
+  const int fixed = (2 * p.pairs + p.rot_panels + KB / 64) * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
+  const int rot_bytes = p.rot_panels * key_panel;
+  p.rot_stages = fixed + 2 * rot_bytes + 2 * p.pairs * 2 * key_panel <= kSmemLimit ? 2 : 1;
+  int ring = (kSmemLimit - fixed - p.rot_stages * rot_bytes) / (2 * key_panel);
+  if (ring > 3 * p.pairs) ring = 3 * p.pairs;
   if (ring > kMaxRing) ring = kMaxRing;
-  if (ring < p.pairs) return kErrTooLarge;
   p.ring = ring;
   p.lookahead = ring >= 2 * p.pairs;
+  return fixed + p.rot_stages * rot_bytes + ring * 2 * key_panel;
+}
+
+template <int HN>
+static bool small_tiles(DecodeParams p) {
+  plan_decode<HN, 128>(p);
+  return !p.lookahead;
+}
+
+template <int HN, int KB>
+static int launch_decode(DecodeParams& p, const void* q, const void* cache, int splits, cudaStream_t st) {
+  const int smem = plan_decode<HN, KB>(p);
+  if (p.ring < p.pairs || smem > kSmemLimit) return kErrTooLarge;
   int cols = 32;
   while (cols < 2 * HN + p.pairs * HN) cols *= 2;
   p.tmem_cols = cols;
@@ -745,17 +768,23 @@ static int launch_decode(DecodeParams& p, const void* q, const void* cache, int 
   CUtensorMap tq, tc, tr;
   int rc;
   if ((rc = map3(&tq, q, row, p.heads, p.b, row, row * p.heads, HN, 1)) != kOk) return rc;
-  if ((rc = map3(&tc, cache, p.rank, p.slots, p.b, row, row * p.slots, kBlk, 1)) != kOk) return rc;
-  if ((rc = map3(&tr, static_cast<const __nv_bfloat16*>(cache) + p.rank, p.rot, p.slots, p.b, row, row * p.slots, kBlk, 1)) != kOk) return rc;
-  const int smem = fixed + p.rot_stages * rot_bytes + ring * kPairBytes;
+  if ((rc = map3(&tc, cache, p.rank, p.slots, p.b, row, row * p.slots, KB, 1)) != kOk) return rc;
+  if ((rc = map3(&tr, static_cast<const __nv_bfloat16*>(cache) + p.rank, p.rot, p.slots, p.b, row, row * p.slots, KB, 1)) != kOk) return rc;
   static bool attr = false;
   if (!attr) {
-    if (cudaFuncSetAttribute(latent_decode_kernel<HN>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit) != cudaSuccess) return kErrDriver;
+    if (cudaFuncSetAttribute(latent_decode_kernel<HN, KB>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit) != cudaSuccess) return kErrDriver;
     attr = true;
   }
   TTB_COUNT_LAUNCH(1);
-  latent_decode_kernel<HN><<<dim3(splits, (p.heads + HN - 1) / HN, p.b), kDecodeThreads, smem, st>>>(tq, tc, tr, p);
+  latent_decode_kernel<HN, KB><<<dim3(splits, (p.heads + HN - 1) / HN, p.b), kDecodeThreads, smem, st>>>(tq, tc, tr, p);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
+}
+
+static DecodeParams decode_shape(int heads, int rank, int rot) {
+  DecodeParams p{};
+  p.heads = heads, p.rank = rank, p.rot = rot;
+  p.pairs = (rank + 127) / 128, p.c_steps = (rank + 15) / 16, p.rot_panels = (rot + 63) / 64, p.rot_steps = (rot + 15) / 16;
+  return p;
 }
 
 }  // namespace latent
@@ -812,13 +841,19 @@ extern "C" int ttb_latent_decode(const void* q, const void* cache, float* o, flo
   using namespace ttb::latent;
   if (b <= 0 || heads <= 0 || slots <= 0 || splits <= 0 || (rank & 7) || (rot & 7) || rank <= 0 || rot <= 0) return kErrBadShape;
   if (rank > 512 || rot > 128) return kErrTooLarge;
-  DecodeParams p{};
-  p.b = b, p.heads = heads, p.rank = rank, p.rot = rot, p.slots = slots, p.scale = scale;
-  p.pairs = (rank + 127) / 128, p.c_steps = (rank + 15) / 16, p.rot_panels = (rot + 63) / 64, p.rot_steps = (rot + 15) / 16;
+  DecodeParams p = decode_shape(heads, rank, rot);
+  p.b = b, p.slots = slots, p.scale = scale;
   p.slot = slot, p.slot_host = slot_host, p.lo = lo, p.lo_row = lo_row, p.hi = hi, p.hi_row = hi_row;
   p.o = o, p.ml = reinterpret_cast<float2*>(ml), p.err = err;
   auto st = static_cast<cudaStream_t>(stream);
-  if (heads <= 16) return launch_decode<16>(p, q, cache, splits, st);
-  const int rc = launch_decode<32>(p, q, cache, splits, st);
-  return rc == kErrTooLarge ? launch_decode<16>(p, q, cache, splits, st) : rc;
+  if (heads <= 16) return small_tiles<16>(p) ? launch_decode<16, 64>(p, q, cache, splits, st) : launch_decode<16, 128>(p, q, cache, splits, st);
+  return small_tiles<32>(p) ? launch_decode<32, 64>(p, q, cache, splits, st) : launch_decode<32, 128>(p, q, cache, splits, st);
+}
+
+// Keys per tile of ttb_latent_decode for these sizes (a key range should not be shorter).
+extern "C" int ttb_latent_decode_tile(int heads, int rank, int rot) {
+  using namespace ttb::latent;
+  if (rank <= 0 || rank > 512 || rot <= 0 || rot > 128) return 128;
+  const DecodeParams p = decode_shape(heads, rank, rot);
+  return (heads <= 16 ? small_tiles<16>(p) : small_tiles<32>(p)) ? 64 : 128;
 }

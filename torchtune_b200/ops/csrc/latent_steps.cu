@@ -3,7 +3,8 @@
 //   latent_prepare     one launch per layer after the input projections: norm of the latent, rotation of the shared key part and of
 //                      the queries' rotated parts, and the write of the latent row into the cache
 //   latent_absorb      q_lat[r, h, :] = W_uk[h]^T q[r, h, :]            (few rows: weight-streaming)
-//   latent_value       out[r, h, :] = (W_uv[h] o_lat[r, h, :]) * sigmoid(gate), combining the split-key partials of the decode kernel
+//   latent_combine     split-key partials of the decode kernel -> latent outputs
+//   latent_value       out[r, h, :] = (W_uv[h] o_lat[r, h, :]) * sigmoid(gate)
 //   latent_attention_any   attention for every size and for fp32 (no tensor cores); queries or heads as rows
 #include <cuda_bf16.h>
 #include <cuda_runtime.h>
@@ -55,7 +56,83 @@ struct PrepareParams {
   int slot_host;
   int s, slots, heads, dim, rot, rot_dims, rank, table_len;
   float eps;
+  int vec;               // bf16 rows that can be read and written 16 bytes at a time
 };
+
+__device__ __forceinline__ void unpack8(const uint4& u, float (&f)[8]) {
+  const __nv_bfloat162* b = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    const float2 t = __bfloat1622float2(b[i]);
+    f[2 * i] = t.x, f[2 * i + 1] = t.y;
+  }
+}
+__device__ __forceinline__ uint4 pack8(const float (&f)[8]) {
+  uint4 u;
+  __nv_bfloat162* b = reinterpret_cast<__nv_bfloat162*>(&u);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) b[i] = __floats2bfloat162_rn(f[2 * i], f[2 * i + 1]);
+  return u;
+}
+// four pairs turned by the angles whose (cos, sin) start at t
+__device__ __forceinline__ uint4 turn8(const uint4& u, const float* t) {
+  float f[8], o[8];
+  unpack8(u, f);
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    o[2 * i] = f[2 * i] * t[2 * i] - f[2 * i + 1] * t[2 * i + 1];
+    o[2 * i + 1] = f[2 * i + 1] * t[2 * i] + f[2 * i] * t[2 * i + 1];
+  }
+  return pack8(o);
+}
+
+// One token, 128 threads: the latent (at most 1024 values) stays in registers between its sum of squares and the scaling, and the
+// queries' rotated parts are fetched before the reduction.
+__device__ __forceinline__ void prepare_row_vec8(const PrepareParams& p, const float* cs, float* scratch, long long row, int bi, int slot) {
+  const int per_head = p.rot >> 3, turned = p.rot_dims >> 3, total = p.heads * per_head;
+  uint4* q = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.q) + row * p.ld_q);
+  const int q_pitch = (p.dim + p.rot) >> 3, q_off = p.dim >> 3, o_pitch = (p.rank + p.rot) >> 3, o_off = p.rank >> 3;
+  uint4* out = p.q_out != nullptr ? reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.q_out) + row * p.heads * (p.rank + p.rot)) : nullptr;
+  int h0 = 0, c0 = 0;
+  uint4 first = make_uint4(0u, 0u, 0u, 0u);
+  if (static_cast<int>(threadIdx.x) < total) {
+    h0 = threadIdx.x / per_head, c0 = threadIdx.x - h0 * per_head;
+    first = q[h0 * q_pitch + q_off + c0];
+  }
+  if (p.kv != nullptr) {
+    const uint4* src = reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.kv) + row * p.ld_kv);
+    const int i = threadIdx.x, n = p.rank >> 3;
+    float f[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    if (i < n) unpack8(src[i], f);
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += f[j] * f[j];
+    ss = warp_sum(ss);
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = ss;
+    __syncthreads();
+    const float rs = 1.f / sqrtf((scratch[0] + scratch[1] + scratch[2] + scratch[3]) / static_cast<float>(p.rank) + p.eps);
+    if (slot >= 0 && slot < p.slots) {
+      uint4* dst = reinterpret_cast<uint4*>(static_cast<__nv_bfloat16*>(p.cache) + (static_cast<long long>(bi) * p.slots + slot) * (p.rank + p.rot));
+      if (i < n) {
+        float g[8];
+        unpack8(reinterpret_cast<const uint4*>(p.kv_gain)[i], g);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) f[j] = f[j] * rs * g[j];
+        dst[i] = pack8(f);
+      }
+      for (int k = threadIdx.x; k < per_head; k += 128) dst[n + k] = k < turned ? turn8(src[n + k], cs + k * 8) : src[n + k];
+    } else if (threadIdx.x == 0) {
+      TTB_NOTE_VIOLATION(latent);
+    }
+  }
+  for (int w = threadIdx.x; w < total; w += 128) {
+    const int h = w == static_cast<int>(threadIdx.x) ? h0 : w / per_head;
+    const int c = w == static_cast<int>(threadIdx.x) ? c0 : w - h * per_head;
+    const uint4 u = w == static_cast<int>(threadIdx.x) ? first : q[h * q_pitch + q_off + c];
+    if (out != nullptr) out[h * o_pitch + o_off + c] = c < turned ? turn8(u, cs + c * 8) : u;
+    else if (c < turned) q[h * q_pitch + q_off + c] = turn8(u, cs + c * 8);
+  }
+}
 
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prepare_kernel(PrepareParams p) {
@@ -73,6 +150,12 @@ __global__ void __launch_bounds__(128) latent_prepare_kernel(PrepareParams p) {
   __syncthreads();
   const int half = p.rot_dims / 2;
 
+  if constexpr (sizeof(T) == 2) {
+    if (p.vec) {
+      prepare_row_vec8(p, cs, scratch, row, bi, slot);
+      return;
+    }
+  }
   if (p.kv != nullptr) {
     const T* src = static_cast<const T*>(p.kv) + row * p.ld_kv;
     const T* gain = static_cast<const T*>(p.kv_gain);
@@ -131,6 +214,10 @@ struct WVec<float, 4> {
     const float4 v = __ldg(reinterpret_cast<const float4*>(p));
     f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
   }
+  static __device__ __forceinline__ void load_shared(const float* p, float (&f)[4]) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+  }
 };
 template <>
 struct WVec<__nv_bfloat16, 4> {
@@ -144,6 +231,7 @@ struct WVec<__nv_bfloat16, 4> {
 template <typename T>
 struct WVec<T, 1> {
   static __device__ __forceinline__ void load(const T* p, float (&f)[1]) { f[0] = to_f(*p); }
+  static __device__ __forceinline__ void load_shared(const T* p, float (&f)[1]) { f[0] = to_f(*p); }
 };
 
 static constexpr int kRows = 8;
@@ -156,20 +244,22 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
   float* sP = sm + kRows * K;      // [8][kRows][32 * VEC]
   const int h = blockIdx.y, r0 = blockIdx.z * kRows;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n = blockIdx.x * 32 * VEC + lane * VEC;
+  const T* wp = w + static_cast<long long>(h) * K * N + n;
+  if (n < N)  // the weights are on their way while the rows are staged
+    for (int k = warp; k < K; k += 8) asm volatile("prefetch.global.L2 [%0];" ::"l"(wp + static_cast<long long>(k) * N));
   for (int t = threadIdx.x; t < kRows * K; t += 256) {
     const int r = t / K, k = t - r * K;
     sA[t] = r0 + r < R ? to_f(a[(r0 + r) * a_row + static_cast<long long>(h) * a_head + k]) : 0.f;
   }
   __syncthreads();
-  const int n = blockIdx.x * 32 * VEC + lane * VEC;
   float acc[kRows][VEC];
 #pragma unroll
   for (int r = 0; r < kRows; ++r)
 #pragma unroll
     for (int v = 0; v < VEC; ++v) acc[r][v] = 0.f;
   if (n < N) {
-    const T* wp = w + static_cast<long long>(h) * K * N + n;
-#pragma unroll 4
+#pragma unroll 8
     for (int k = warp; k < K; k += 8) {
       float f[VEC];
       WVec<T, VEC>::load(wp + static_cast<long long>(k) * N, f);
@@ -197,86 +287,109 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
   }
 }
 
-// ------------------------------------------------------------------------------- value projection: contraction along weight rows
-// o [splits, R, heads, K] fp32 with ml [splits, R, heads] (log2-domain maximum, sum).  Each CTA first combines the partials of its rows
-// in shared memory, then out[r, h, n] = (sum_k c[r, h, k] * w[h * N + n, k]) * sigmoid(gate[r, h * N + n]).
-static constexpr int kValueCols = 32;
-
-__device__ __forceinline__ void combine_rows(const float* __restrict__ o, const float2* __restrict__ ml, float* __restrict__ dst, int dst_pitch, int splits, int R,
-                                             int heads, int h, int r0, int n_rows, int K, float* wts) {
-  // wts [n_rows][splits]: exp2(m_s - m) / sum
-  if (static_cast<int>(threadIdx.x) < n_rows) {
-    const int r = threadIdx.x;
-    float m = -INFINITY, l = 0.f;
-    if (r0 + r < R) {
-      for (int s = 0; s < splits; ++s) {
-        const float2 v = ml[(static_cast<long long>(s) * R + r0 + r) * heads + h];
-        if (v.y > 0.f) m = fmaxf(m, v.x);
-      }
-      for (int s = 0; s < splits; ++s) {
-        const float2 v = ml[(static_cast<long long>(s) * R + r0 + r) * heads + h];
-        if (v.y > 0.f) l += v.y * exp2f(v.x - m);
-      }
-    }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float2 v = r0 + r < R ? ml[(static_cast<long long>(s) * R + r0 + r) * heads + h] : make_float2(0.f, 0.f);
-      wts[r * splits + s] = v.y > 0.f ? exp2f(v.x - m) * inv : 0.f;
-    }
-  }
-  __syncthreads();
-  for (int t = threadIdx.x; t < n_rows * K; t += blockDim.x) {
-    const int r = t / K, k = t - r * K;
-    float acc = 0.f;
-    if (r0 + r < R) {
-      const float* src = o + (static_cast<long long>(r0 + r) * heads + h) * K + k;
-      const long long pitch = static_cast<long long>(R) * heads * K;
-#pragma unroll 4
-      for (int s = 0; s < splits; ++s) {
-        const float wt = wts[r * splits + s];
-        if (wt != 0.f) acc += wt * src[s * pitch];  // a split without keys has written nothing
-      }
-    }
-    dst[r * dst_pitch + k] = acc;
-  }
-  __syncthreads();
+// ------------------------------------------------------------------------------- split-key partials
+// o [splits, R, heads, K] fp32 with ml [splits, R, heads] (log2-domain maximum, sum) -> the normalised rows, [R, heads, K] fp32 or
+// head-major [heads, R, K] bf16 (the row order of a grouped GEMM whose groups are heads).  One CTA per (row, head, 128 columns).
+__device__ __forceinline__ float warp_max_of(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
+  return v;
 }
 
-template <typename T, int VEC>
-__global__ void __launch_bounds__(256) latent_value_kernel(const float* __restrict__ o, const float2* __restrict__ ml, const T* __restrict__ w,
-                                                           const T* __restrict__ gate, long long gate_ld, T* __restrict__ out, int splits, int R, int heads, int K,
-                                                           int N) {
-  extern __shared__ float sm[];
-  float* sA = sm;                 // [kRows][K]
-  float* wts = sm + kRows * K;    // [kRows][splits]
-  const int h = blockIdx.y, r0 = blockIdx.z * kRows;
-  const int n_rows = min(kRows, R - r0);
-  combine_rows(o, ml, sA, K, splits, R, heads, h, r0, n_rows, K, wts);
-  for (int t = n_rows * K + threadIdx.x; t < kRows * K; t += 256) sA[t] = 0.f;
+template <bool HEAD_MAJOR>
+__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits, int R,
+                                                             int heads, int K) {
+  extern __shared__ float wts[];  // [splits]: exp2(m_s - m) / sum, 0 for a split without keys (which has written nothing)
+  const int r = blockIdx.x, h = blockIdx.y;
+  const long long rh = static_cast<long long>(r) * heads + h, RH = static_cast<long long>(R) * heads;
+  if (threadIdx.x < 32) {
+    float m = -INFINITY, l = 0.f;
+    for (int s = threadIdx.x; s < splits; s += 32) {
+      const float2 v = ml[s * RH + rh];
+      if (v.y > 0.f) {
+        const float m_new = fmaxf(m, v.x);
+        l = l * exp2f(m - m_new) + v.y * exp2f(v.x - m_new);  // m = -inf: the first factor is 0
+        m = m_new;
+      }
+    }
+    const float top = warp_max_of(m);
+    l = warp_sum(m == -INFINITY ? 0.f : l * exp2f(m - top));
+    const float inv = l > 0.f ? 1.f / l : 0.f;
+    for (int s = threadIdx.x; s < splits; s += 32) {
+      const float2 v = ml[s * RH + rh];
+      wts[s] = v.y > 0.f ? exp2f(v.x - top) * inv : 0.f;
+    }
+  }
   __syncthreads();
+  const int k = blockIdx.z * 128 + threadIdx.x;
+  if (k < K) {
+    float acc = 0.f;
+    const float* src = o + rh * K + k;
+#pragma unroll 16
+    for (int s = 0; s < splits; ++s) {
+      const float v = src[s * RH * K];  // loaded in any case, so the loads of many ranges are in flight together
+      acc += wts[s] != 0.f ? wts[s] * v : 0.f;
+    }
+    if constexpr (HEAD_MAJOR) static_cast<__nv_bfloat16*>(out)[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(acc);
+    else static_cast<float*>(out)[rh * K + k] = acc;
+  }
+}
+
+// ------------------------------------------------------------------------------- value projection: contraction along weight rows
+// out[r, h, n] = (sum_k o[r, h, k] * w[h * N + n, k]) / l[r, h] * sigmoid(gate[r, h * N + n]); ml (of one split) == nullptr: l = 1.
+static constexpr int kValueCols = 16;
+
+template <typename T, int VEC, int ROWS>
+__global__ void __launch_bounds__(256) latent_value_kernel(const float* __restrict__ o, const float2* __restrict__ ml, const T* __restrict__ w,
+                                                           const T* __restrict__ gate, long long gate_ld, T* __restrict__ out, int R, int heads, int K, int N) {
+  extern __shared__ __align__(16) float sA[];  // [ROWS][K]
+  const int h = blockIdx.y, r0 = blockIdx.z * ROWS;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int c = warp; c < kValueCols; c += 8) {
-    const int n = blockIdx.x * kValueCols + c;
-    if (n >= N) break;
-    const T* wp = w + (static_cast<long long>(h) * N + n) * K;
-    float acc[kRows];
+  const int n0 = blockIdx.x * kValueCols + warp * 2;
+  const T* wp = w + (static_cast<long long>(h) * N + n0) * K;
 #pragma unroll
-    for (int r = 0; r < kRows; ++r) acc[r] = 0.f;
+  for (int c = 0; c < 2; ++c)
+    if (n0 + c < N)
+      for (int k = lane * (128 / static_cast<int>(sizeof(T))); k < K; k += 32 * (128 / static_cast<int>(sizeof(T))))
+        asm volatile("prefetch.global.L2 [%0];" ::"l"(wp + static_cast<long long>(c) * K + k));
+  for (int t = threadIdx.x; t < ROWS * K; t += 256) {
+    const int r = t / K, k = t - r * K;
+    float v = 0.f;
+    if (r0 + r < R) {
+      const long long rh = static_cast<long long>(r0 + r) * heads + h;
+      float inv = 1.f;
+      if (ml != nullptr) {
+        const float l = ml[rh].y;
+        inv = l > 0.f ? 1.f / l : 0.f;
+      }
+      v = inv == 0.f ? 0.f : o[rh * K + k] * inv;
+    }
+    sA[t] = v;
+  }
+  __syncthreads();
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+    const int n = n0 + c;
+    if (n >= N) break;
+    float acc[ROWS];
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
 #pragma unroll 4
     for (int k = lane * VEC; k < K; k += 32 * VEC) {
       float f[VEC];
-      WVec<T, VEC>::load(wp + k, f);
+      WVec<T, VEC>::load(wp + static_cast<long long>(c) * K + k, f);
 #pragma unroll
-      for (int r = 0; r < kRows; ++r)
+      for (int r = 0; r < ROWS; ++r) {
+        float a[VEC];
+        WVec<float, VEC>::load_shared(sA + r * K + k, a);
 #pragma unroll
-        for (int v = 0; v < VEC; ++v) acc[r] += sA[r * K + k + v] * f[v];
+        for (int v = 0; v < VEC; ++v) acc[r] += a[v] * f[v];
+      }
     }
 #pragma unroll
-    for (int r = 0; r < kRows; ++r) acc[r] = warp_sum(acc[r]);
-    if (lane == 0) {
-#pragma unroll
-      for (int r = 0; r < kRows; ++r) {
-        if (r >= n_rows) continue;
+    for (int r = 0; r < ROWS; ++r) {
+      acc[r] = warp_sum(acc[r]);
+      if (lane == r && r0 + r < R) {
         const long long col = static_cast<long long>(h) * N + n;
         float v = acc[r];
         if (gate != nullptr) v *= sigmoid_as<T>(to_f(gate[(r0 + r) * gate_ld + col]));
@@ -284,17 +397,6 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const float* __restri
       }
     }
   }
-}
-
-// Combined latent outputs only, head-major [heads, R, K] (bf16): the row order of a grouped GEMM whose groups are heads.
-__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, __nv_bfloat16* __restrict__ out, int splits,
-                                                             int R, int heads, int K) {
-  extern __shared__ float sm[];
-  float* row = sm;
-  float* wts = sm + K;
-  const int r = blockIdx.x, h = blockIdx.y;
-  combine_rows(o, ml, row, K, splits, R, heads, h, r, 1, K, wts);
-  for (int k = threadIdx.x; k < K; k += blockDim.x) out[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(row[k]);
 }
 
 // x [heads, R, N] head-major -> out [R, heads * N] with the gate applied; and the way back in for the queries (copy of the unrotated
@@ -482,21 +584,26 @@ static int launch_absorb(const void* a, long long a_row, int a_head, const void*
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 
-template <typename T>
-static int launch_value(const float* o, const float* ml, const void* w, const void* gate, long long gate_ld, void* out, int splits, int R, int heads, int K, int N,
-                        cudaStream_t st) {
-  const bool vec = K % 4 == 0 && !(reinterpret_cast<uintptr_t>(w) & 15);
-  const int smem = (kRows * K + kRows * splits) * 4;
-  static int g4 = 0, g1 = 0;
-  if (!(vec ? allow_smem(latent_value_kernel<T, 4>, smem, g4) : allow_smem(latent_value_kernel<T, 1>, smem, g1))) return kErrTooLarge;
-  const dim3 grid((N + kValueCols - 1) / kValueCols, heads, (R + kRows - 1) / kRows);
-  auto mlp = reinterpret_cast<const float2*>(ml);
+template <typename T, int VEC, int ROWS>
+static int launch_value_rows(const float* o, const float2* ml, const void* w, const void* gate, long long gate_ld, void* out, int R, int heads, int K, int N,
+                             cudaStream_t st) {
+  const int smem = ROWS * K * 4;
+  static int granted = 0;
+  if (!allow_smem(latent_value_kernel<T, VEC, ROWS>, smem, granted)) return kErrTooLarge;
   TTB_COUNT_LAUNCH(1);
-  if (vec)
-    latent_value_kernel<T, 4><<<grid, 256, smem, st>>>(o, mlp, static_cast<const T*>(w), static_cast<const T*>(gate), gate_ld, static_cast<T*>(out), splits, R, heads, K, N);
-  else
-    latent_value_kernel<T, 1><<<grid, 256, smem, st>>>(o, mlp, static_cast<const T*>(w), static_cast<const T*>(gate), gate_ld, static_cast<T*>(out), splits, R, heads, K, N);
+  latent_value_kernel<T, VEC, ROWS><<<dim3((N + kValueCols - 1) / kValueCols, heads, (R + ROWS - 1) / ROWS), 256, smem, st>>>(
+      o, ml, static_cast<const T*>(w), static_cast<const T*>(gate), gate_ld, static_cast<T*>(out), R, heads, K, N);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
+}
+
+template <typename T>
+static int launch_value(const float* o, const float* ml, const void* w, const void* gate, long long gate_ld, void* out, int R, int heads, int K, int N,
+                        cudaStream_t st) {
+  auto m = reinterpret_cast<const float2*>(ml);
+  if (K % 4 || (reinterpret_cast<uintptr_t>(w) & 15)) return launch_value_rows<T, 1, kRows>(o, m, w, gate, gate_ld, out, R, heads, K, N, st);
+  if (R == 1) return launch_value_rows<T, 4, 1>(o, m, w, gate, gate_ld, out, R, heads, K, N, st);
+  if (R <= 4) return launch_value_rows<T, 4, 4>(o, m, w, gate, gate_ld, out, R, heads, K, N, st);
+  return launch_value_rows<T, 4, kRows>(o, m, w, gate, gate_ld, out, R, heads, K, N, st);
 }
 
 }  // namespace latent
@@ -511,7 +618,10 @@ extern "C" int ttb_latent_prepare(const void* kv, long long ld_kv, const void* k
                                   int table_len, float eps, int wide, void* stream) {
   if (rows <= 0 || s <= 0 || rows % s || heads <= 0 || rot_dims < 0 || (rot_dims & 1) || rot_dims > rot || table_len <= 0) return kErrBadShape;
   if (kv != nullptr && (kv_gain == nullptr || cache == nullptr || slots <= 0)) return kErrBadShape;
-  PrepareParams p{kv, ld_kv, kv_gain, q, ld_q, q_out, cache, table, pos, slot, slot_host, s, slots, heads, dim, rot, rot_dims, rank, table_len, eps};
+  PrepareParams p{kv, ld_kv, kv_gain, q, ld_q, q_out, cache, table, pos, slot, slot_host, s, slots, heads, dim, rot, rot_dims, rank, table_len, eps, 0};
+  const uintptr_t at = reinterpret_cast<uintptr_t>(kv) | reinterpret_cast<uintptr_t>(kv_gain) | reinterpret_cast<uintptr_t>(q) | reinterpret_cast<uintptr_t>(q_out) |
+                       reinterpret_cast<uintptr_t>(cache);
+  p.vec = !wide && !(at & 15) && !((ld_kv | ld_q | dim | rot | rot_dims | rank) & 7) && rank <= 1024;
   auto st = static_cast<cudaStream_t>(stream);
   TTB_COUNT_LAUNCH(1);
   if (wide) latent_prepare_kernel<float><<<rows, 128, rot_dims * 4, st>>>(p);
@@ -528,21 +638,23 @@ extern "C" int ttb_latent_absorb(const void* a, long long a_row, int a_head, con
               : launch_absorb<__nv_bfloat16>(a, a_row, a_head, w, out, out_row, out_head, rows, heads, K, N, st);
 }
 
-// o [splits, rows, heads, K] / ml [splits, rows, heads, 2] fp32, w [heads*N, K]; out [rows, heads*N]
-extern "C" int ttb_latent_value(const float* o, const float* ml, const void* w, const void* gate, long long gate_ld, void* out, int splits, int rows, int heads, int K,
-                                int N, int wide, void* stream) {
-  if (rows <= 0 || heads <= 0 || K <= 0 || N <= 0 || splits <= 0) return kErrBadShape;
+// o [rows, heads, K] fp32, w [heads*N, K]; out [rows, heads*N].  ml [rows, heads, 2] (of one split) divides by the sum, nullptr: o is normalised.
+extern "C" int ttb_latent_value(const float* o, const float* ml, const void* w, const void* gate, long long gate_ld, void* out, int rows, int heads, int K, int N,
+                                int wide, void* stream) {
+  if (rows <= 0 || heads <= 0 || K <= 0 || N <= 0) return kErrBadShape;
   auto st = static_cast<cudaStream_t>(stream);
-  return wide ? launch_value<float>(o, ml, w, gate, gate_ld, out, splits, rows, heads, K, N, st)
-              : launch_value<__nv_bfloat16>(o, ml, w, gate, gate_ld, out, splits, rows, heads, K, N, st);
+  return wide ? launch_value<float>(o, ml, w, gate, gate_ld, out, rows, heads, K, N, st)
+              : launch_value<__nv_bfloat16>(o, ml, w, gate, gate_ld, out, rows, heads, K, N, st);
 }
 
-// bf16, head-major [heads, rows, K]
-extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, int splits, int rows, int heads, int K, void* stream) {
-  if (rows <= 0 || heads <= 0 || K <= 0 || splits <= 0 || (K + splits) * 4 > 48 * 1024) return kErrBadShape;
+// [rows, heads, K] fp32, or (head_major) [heads, rows, K] bf16
+extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, int splits, int rows, int heads, int K, int head_major, void* stream) {
+  if (rows <= 0 || heads <= 0 || K <= 0 || splits <= 0 || splits > 8192) return kErrBadShape;
+  auto st = static_cast<cudaStream_t>(stream);
+  auto m = reinterpret_cast<const float2*>(ml);
   TTB_COUNT_LAUNCH(1);
-  latent_combine_kernel<<<dim3(rows, heads), 128, (K + splits) * 4, static_cast<cudaStream_t>(stream)>>>(o, reinterpret_cast<const float2*>(ml),
-                                                                                                       static_cast<__nv_bfloat16*>(out), splits, rows, heads, K);
+  if (head_major) latent_combine_kernel<true><<<dim3(rows, heads, (K + 127) / 128), 128, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
+  else latent_combine_kernel<false><<<dim3(rows, heads, (K + 127) / 128), 128, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 

@@ -92,13 +92,13 @@ def decode_supported(q: torch.Tensor, rank: int, rot: int) -> bool:
     return q.dtype == torch.bfloat16 and rank % 8 == 0 and rot % 8 == 0 and rank <= 512 and rot <= 128
 
 
-def split_count(b: int, heads: int, keys: int) -> int:
-    """Key ranges per (batch row, head group): enough CTAs for one per SM, at least one 128-key tile each."""
+def split_count(b: int, heads: int, rank: int, rot: int, keys: int) -> int:
+    """Key ranges per (batch row, head group): enough CTAs for one per SM, at least one tile of keys each."""
     global _SMS
     if _SMS is None:
         _SMS = torch.cuda.get_device_properties(torch.cuda.current_device()).multi_processor_count
     groups = 1 if heads <= 16 else -(-heads // 32)
-    return max(1, min(-(-keys // 128), _SMS // (b * groups)))
+    return max(1, min(-(-keys // lib().ttb_latent_decode_tile(heads, rank, rot)), _SMS // (b * groups)))
 
 
 def absorb(q: torch.Tensor, w_uk: torch.Tensor, q_lat: torch.Tensor, *, heads: int, dim: int, rot: int, rank: int) -> None:
@@ -135,7 +135,7 @@ def decode(q_lat: torch.Tensor, buf: torch.Tensor, *, rank: int, rot: int, scale
     assert width == rank + rot and buf.shape[0] >= b and buf.shape[2] == width and buf.is_contiguous() and buf.dtype == q_lat.dtype and q_lat.is_contiguous()
     slots = buf.shape[1]
     if decode_supported(q_lat, rank, rot):
-        splits = split_count(b, heads, keys)
+        splits = split_count(b, heads, rank, rot, keys)
         o = torch.empty(splits, b, heads, rank, dtype=torch.float32, device=q_lat.device)
         ml = torch.empty(splits, b, heads, 2, dtype=torch.float32, device=q_lat.device)
         check(lib().ttb_latent_decode(q_lat.data_ptr(), buf.data_ptr(), o.data_ptr(), ml.data_ptr(), b, heads, rank, rot, slots, splits, _p(slot), int(slot_host), _p(bounds.lo),
@@ -160,11 +160,15 @@ def value(o: torch.Tensor, ml: torch.Tensor, w_uv: torch.Tensor, gate: Optional[
         from ._cuda import _grouped_gemm
 
         lat = torch.empty(heads * rows, rank, dtype=torch.bfloat16, device=o.device)
-        check(lib().ttb_latent_combine(o.data_ptr(), ml.data_ptr(), lat.data_ptr(), splits, rows, heads, rank, stream_ptr()), "latent_combine")
+        check(lib().ttb_latent_combine(o.data_ptr(), ml.data_ptr(), lat.data_ptr(), splits, rows, heads, rank, 1, stream_ptr()), "latent_combine")
         y = _grouped_gemm(lat, w_uv.view(heads, vdim, rank), _head_counts(heads, rows, o.device), b_mn=False)
         check(lib().ttb_latent_gate_rows(y.data_ptr(), _p(gate), gate_ld, out.data_ptr(), rows, heads, vdim, stream_ptr()), "latent_gate_rows")
         return out
-    check(lib().ttb_latent_value(o.data_ptr(), ml.data_ptr(), w_uv.data_ptr(), _p(gate), gate_ld, out.data_ptr(), splits, rows, heads, rank, vdim, _wide(w_uv), stream_ptr()), "latent_value")
+    if splits > 1:
+        o1 = torch.empty(rows, heads, rank, dtype=torch.float32, device=o.device)
+        check(lib().ttb_latent_combine(o.data_ptr(), ml.data_ptr(), o1.data_ptr(), splits, rows, heads, rank, 0, stream_ptr()), "latent_combine")
+        o, ml = o1, None
+    check(lib().ttb_latent_value(o.data_ptr(), _p(ml), w_uv.data_ptr(), _p(gate), gate_ld, out.data_ptr(), rows, heads, rank, vdim, _wide(w_uv), stream_ptr()), "latent_value")
     return out
 
 

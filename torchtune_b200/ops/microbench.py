@@ -7,6 +7,7 @@
     python -m torchtune_b200.ops.microbench adamw8bit --numel 268435456
     python -m torchtune_b200.ops.microbench gate_up --tokens 8192 --dim 4096 --hidden 14336
     python -m torchtune_b200.ops.microbench comm --world 8 --numel 268435456             (peer-memory kernels, ranks emulated on one GPU)
+    python -m torchtune_b200.ops.microbench latent --heads 16 --rank 512       (latent attention beside grouped-query attention)
     python -m torchtune_b200.ops.microbench suite --tokens 8192      (norm, RoPE, SwiGLU, loss, embedding, LoRA, grouped GEMM, NF4, offload copies)
 
 Each command prints one JSON line: median milliseconds over ``--iters`` launches (an L2 flush
@@ -137,6 +138,108 @@ def bench_attention(args, flush):
     t = _time(lambda: torch.autograd.grad(out, (q, k, v), go, retain_graph=True), args.iters, args.warmup, flush)
     res.update(bwd_ms=t, bwd_tflops=2.5 * fwd_flops / t / 1e9)
     return res
+
+
+def _time_captured(make, iters: int, total_bytes: float) -> float:
+    """Median milliseconds of one call out of a CUDA graph that runs ``make(i)()`` for enough independent inputs ``i`` to exceed L2."""
+    copies = int(max(4, min(64, 400e6 // max(total_bytes, 1.0) + 1)))
+    fns = [make(i) for i in range(copies)]
+    keep = [fn() for fn in fns]
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        keep = [fn() for fn in fns]
+    times = []
+    for _ in range(iters + 2):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        e0.record()
+        graph.replay()
+        e1.record()
+        torch.cuda.synchronize()
+        times.append(e0.elapsed_time(e1) / copies)
+    del keep
+    times = sorted(times[2:])
+    return times[len(times) // 2]
+
+
+def bench_latent(args, flush):
+    """Kernels of latent attention and the 32-bit residual stream beside the like kernels of a grouped-query decoder of equal width, heads and
+    context: one JSON line per kernel with milliseconds and the achieved TFLOP/s or GB/s of its algorithmic work."""
+    from . import latent, linear, rms_norm
+    from ._cuda_attention import attention
+    from .mask import AttentionMask
+
+    H, d, r, dv, rank, D = args.heads, args.head_dim, args.rot, args.head_dim, args.rank, args.dim
+    hk = max(1, H // 4)
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    it, wu = args.iters, args.warmup
+    rows = []
+
+    def emit(op, ms, **kw):
+        row = {"op": op, "ms": round(ms, 5), **{k: (round(v, 1) if isinstance(v, float) else v) for k, v in kw.items()}}
+        rows.append(row)
+        print(json.dumps(row), flush=True)
+
+    with torch.no_grad():
+        for b, s in ((1, args.seq), (4, args.seq // 4)):
+            q, kv = torch.randn(b * s, H * (d + r), **bf), torch.randn(b * s, H * (d + dv), **bf)
+            kn, v = kv.split([H * d, H * dv], dim=1)
+            buf, g = torch.randn(b, s, rank + r, **bf), torch.randn(b * s, H * dv, **bf)
+            pairs = b * H * s * (s + 1) / 2
+            t = _time(lambda: latent.prefill(q, kn, v, buf, g, b=b, s=s, sk=s, slot0=0, heads=H, dim=d, rot=r, vdim=dv, rank=rank, scale=0.07, bounds=latent.Bounds()), it, wu, flush)
+            emit("latent_prefill", t, batch=b, seq=s, tflops=2 * pairs * (d + r + dv) / t / 1e9)
+            qa, ka, va = torch.randn(b, s, H, d, **bf), torch.randn(b, s, hk, d, **bf), torch.randn(b, s, hk, d, **bf)
+            t = _time(lambda: attention(qa, ka, va, AttentionMask(causal=True), None, 0.0), it, wu, flush)
+            emit("gqa_prefill", t, batch=b, seq=s, tflops=4 * pairs * d / t / 1e9)
+        for b, keys in ((1, 8192), (8, 4096), (32, 4096), (128, 2048)):
+            nbytes = b * keys * (rank + r) * 2.0
+            bufs = [torch.randn(b, keys, rank + r, **bf) for _ in range(int(max(4, min(64, 400e6 // nbytes + 1))))]
+            q = torch.randn(b, H, rank + r, **bf)
+            t = _time_captured(lambda i: lambda: latent.decode(q, bufs[i % len(bufs)], rank=rank, rot=r, scale=0.05, slot=None, slot_host=keys - 1, bounds=latent.Bounds(), keys=keys), it, nbytes)
+            emit("latent_decode", t, batch=b, keys=keys, gbs=nbytes / t / 1e6, tflops=2.0 * b * keys * H * (2 * rank + r) / t / 1e9)
+            nbytes = b * keys * hk * d * 4.0
+            n = int(max(4, min(64, 400e6 // nbytes + 1)))
+            ks, vs = [torch.randn(b, keys, hk, d, **bf) for _ in range(n)], [torch.randn(b, keys, hk, d, **bf) for _ in range(n)]
+            qa = torch.randn(b, 1, H, d, **bf)
+            m = AttentionMask(causal=False, bool_mask=torch.ones(b, 1, keys, dtype=torch.bool, device="cuda"))
+            t = _time_captured(lambda i: lambda: attention(qa, ks[i % n], vs[i % n], m, None, 0.0), it, nbytes)
+            emit("gqa_decode", t, batch=b, keys=keys, gbs=nbytes / t / 1e6)
+            del bufs, ks, vs
+        for T in (1, 16, 64, 8192):
+            nbytes = T * D * 12.0
+            x, y, w = torch.randn(T, D, device="cuda"), torch.randn(T, D, **bf), torch.randn(D, **bf)
+            t = _time_captured(lambda i: lambda: latent.residual_norm(x, y, w, w, 1e-6, 0.5, 1.0), it, nbytes) if T < 1024 else _time(lambda: latent.residual_norm(x, y, w, w, 1e-6, 0.5, 1.0), it, wu, flush)
+            emit("residual_norm", t, rows=T, gbs=nbytes / t / 1e6)
+            xb = torch.randn(T, D, **bf)
+            t = _time_captured(lambda i: lambda: rms_norm(xb, w, 1e-6), it, T * D * 4.0) if T < 1024 else _time(lambda: rms_norm(xb, w, 1e-6), it, wu, flush)
+            emit("rms_norm", t, rows=T, gbs=T * D * 4.0 / t / 1e6)
+        table = torch.randn(8192, r // 2, 2, device="cuda")
+        for T in (1, 16, 64, 8192):
+            qkv, gain, buf = torch.randn(T, H * (d + r) + rank + r, **bf), torch.randn(rank, **bf), torch.zeros(1 if T > 64 else T, T if T > 64 else 8, rank + r, **bf)
+            q, kv = qkv.split([H * (d + r), rank + r], dim=1)
+            run = lambda: latent.prepare(q, kv, gain, buf, table, None, s=T if T > 64 else 1, slot=None, slot_host=0, heads=H, dim=d, rot=r, rot_dims=r, rank=rank, eps=1e-6)  # noqa: E731
+            nbytes = T * (2.0 * H * r + 2 * (rank + r)) * 2
+            t = _time(run, it, wu, flush) if T > 64 else _time_captured(lambda i: run, it, nbytes)
+            emit("latent_prepare", t, rows=T, gbs=nbytes / t / 1e6)
+        for T in (1, 8, 16, 64, 256):
+            nbytes = H * d * rank * 2.0
+            n = int(max(4, min(64, 400e6 // nbytes + 1)))
+            ws = [torch.randn(H * d, rank, **bf) for _ in range(n)]
+            q, ql, g = torch.randn(T, H * (d + r), **bf), torch.empty(T, H, rank + r, **bf), torch.randn(T, H * dv, **bf)
+            t = _time_captured(lambda i: lambda: latent.absorb(q, ws[i % n], ql, heads=H, dim=d, rot=r, rank=rank), it, nbytes)
+            emit("latent_absorb", t, rows=T, gbs=nbytes / t / 1e6, tflops=2.0 * T * H * d * rank / t / 1e9)
+            splits = latent.split_count(T, H, rank, r, 4096)
+            o, ml = torch.randn(splits, T, H, rank, device="cuda"), torch.ones(splits, T, H, 2, device="cuda")
+            t = _time_captured(lambda i: lambda: latent.value(o, ml, ws[i % n], g, vdim=dv), it, nbytes)
+            emit("latent_value", t, rows=T, splits=splits, gbs=(nbytes + o.numel() * 4.0) / t / 1e6, tflops=2.0 * T * H * d * rank / t / 1e9)
+            wq = [torch.randn(H * d, D, **bf) for _ in range(8)]
+            xq = torch.randn(T, D, **bf)
+            t = _time_captured(lambda i: lambda: linear(xq, wq[i % 8]), it, H * d * D * 2.0)
+            emit("linear_q (gqa)", t, rows=T, gbs=H * d * D * 2.0 / t / 1e6)
+            wj = [torch.randn(H * (d + r) + rank + r + H * dv, D, **bf) for _ in range(8)]
+            t = _time_captured(lambda i: lambda: linear(xq, wj[i % 8]), it, wj[0].numel() * 2.0)
+            emit("linear_joined", t, rows=T, gbs=wj[0].numel() * 2.0 / t / 1e6)
+    return {"op": "latent", "heads": H, "kernels": len(rows)}
 
 
 def bench_rmsnorm(args, flush):
@@ -449,13 +552,20 @@ def main() -> None:
     co = sub.add_parser("comm")
     co.add_argument("--world", type=int, default=8)
     co.add_argument("--numel", type=int, default=1 << 28)
+    la = sub.add_parser("latent")
+    la.add_argument("--heads", type=int, default=16)
+    la.add_argument("--head-dim", type=int, default=128)
+    la.add_argument("--rot", type=int, default=64)
+    la.add_argument("--rank", type=int, default=512)
+    la.add_argument("--dim", type=int, default=2048)
+    la.add_argument("--seq", type=int, default=8192)
     su = sub.add_parser("suite")
     su.add_argument("--tokens", type=int, default=8192)
     args = ap.parse_args()
     from ._lib import check_device_errors
 
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
-    fn = {"gemm": bench_gemm, "gemm_fp8": bench_gemm_fp8, "gemm_mxfp8": bench_gemm_mxfp8, "attention": bench_attention, "rmsnorm": bench_rmsnorm, "adamw": bench_adamw, "adamw8bit": bench_adamw8bit, "gate_up": bench_gate_up, "comm": bench_comm, "suite": bench_suite}[args.op]
+    fn = {"gemm": bench_gemm, "gemm_fp8": bench_gemm_fp8, "gemm_mxfp8": bench_gemm_mxfp8, "attention": bench_attention, "rmsnorm": bench_rmsnorm, "adamw": bench_adamw, "adamw8bit": bench_adamw8bit, "gate_up": bench_gate_up, "comm": bench_comm, "latent": bench_latent, "suite": bench_suite}[args.op]
     res = fn(args, flush)
     check_device_errors()
     print(json.dumps(res), flush=True)
