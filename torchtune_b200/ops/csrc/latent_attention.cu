@@ -29,14 +29,6 @@ using namespace attn;
 
 __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + __expf(-z)); }
 
-// Up to four contraction steps (of 16 columns) of one pair of 64-column K-major panels.  `da` / `db` describe the panels' first steps; a step
-// further is 32 bytes, i.e. 2 in the descriptors' address fields, so the issuing thread spends one addition per operand.
-__device__ __forceinline__ void umma_panel(uint32_t d, uint64_t da, uint64_t db, int steps, uint32_t idesc, bool accumulate) {
-#pragma unroll
-  for (int k = 0; k < 4; ++k)
-    if (k < steps) umma_f16(d, da + 2 * k, db + 2 * k, idesc, accumulate || k > 0);
-}
-
 // ===================================================================================== prefill
 struct PrefillParams {
   int b, s, sk, heads;
@@ -189,9 +181,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       }
       tc_fence_after();
       if (lane == 0) {
-        uint64_t dq = desc_kmajor(aQ + x * q_bytes, 0), dk = desc_kmajor(aK + st * q_bytes, 0);
-        for (int c = 0; c < p.dim_panels; ++c, dq += kPanelBytes >> 4, dk += kPanelBytes >> 4) umma_panel(tS[x], dq, dk, p.dim_steps - 4 * c, idesc_s, c > 0);
-        for (int c = 0; c < p.rot_panels; ++c, dq += kPanelBytes >> 4, dk += kPanelBytes >> 4) umma_panel(tS[x], dq, dk, p.rot_steps - 4 * c, idesc_s, true);
+        const uint32_t q_base = aQ + x * q_bytes, k_base = aK + st * q_bytes;
+        for (int k = 0; k < p.dim_steps; ++k) umma_f16(tS[x], desc_kmajor(q_base, k), desc_kmajor(k_base, k), idesc_s, k != 0);
+        const uint32_t off = p.dim_panels * kPanelBytes;
+        for (int k = 0; k < p.rot_steps; ++k) umma_f16(tS[x], desc_kmajor(q_base + off, k), desc_kmajor(k_base + off, k), idesc_s, 1);
         umma_commit(&s_full[x]);
         const bool other_later = (x == 0) && active(1, j);  // tile 1 issues its S(j) after tile 0's
         if (!other_later) umma_commit(&k_empty[st]);
@@ -401,7 +394,7 @@ struct DecodeParams {
   int c_steps, rot_panels, rot_steps;
   int ring;        // 32 KB slots for pieces
   int rot_stages;
-  int lookahead;   // ring holds two tiles: the next scores are issued before this tile's outputs
+  int lookahead;   // the ring holds two tiles: loads and scores of the next run beside this tile's outputs
   int tmem_cols;
   float scale;
   const int* slot;  // device: cache slot of the newest token (nullptr: slot_host)
@@ -417,7 +410,7 @@ struct DecodeParams {
 
 static constexpr int kDecodeThreads = 256;
 static constexpr int kMaxRing = 12;
-static constexpr int kDecodeBarriers = 2 * kMaxRing + 4 + 4 + 3;
+static constexpr int kDecodeBarriers = 2 * kMaxRing + 4 + 4 + 5;
 
 __device__ __forceinline__ float warp_max(float v) {
   float r;
@@ -439,6 +432,14 @@ __device__ __forceinline__ bool group_any(bool v) {
 }
 __device__ __forceinline__ void group_sync() { asm volatile("barrier.cta.sync 1, 128;" ::: "memory"); }
 
+// Up to four contraction steps (of 16 columns) of one pair of 64-column K-major panels.  `da` / `db` describe the panels' first steps; a step
+// further is 32 bytes, i.e. 2 in the descriptors' address fields, so the issuing thread spends one addition per operand.
+__device__ __forceinline__ void umma_panel(uint32_t d, uint64_t da, uint64_t db, int steps, uint32_t idesc, bool accumulate) {
+#pragma unroll
+  for (int k = 0; k < 4; ++k)
+    if (k < steps) umma_f16(d, da + 2 * k, db + 2 * k, idesc, accumulate || k > 0);
+}
+
 template <int HN>
 __device__ __forceinline__ void tmem_ld_heads(uint32_t addr, uint32_t (&v)[HN]) {
   if constexpr (HN == 16) tmem_ld_32x16(addr, v);
@@ -451,20 +452,19 @@ __device__ __forceinline__ void tmem_st_heads(uint32_t addr, const uint32_t (&v)
 }
 
 // HN: heads per CTA (16 or 32).  KB: keys per tile.  A wide latent leaves room for one and a bit 128-key tiles; tiles of 64 keys are then
-// double-buffered instead.  Their score MMA still has 128 rows: the upper 64 read whatever follows the panel in shared memory (always
-// inside the allocation) and are never looked at.
+// double-buffered instead.  The 64 rows of such a score tile land in the first 16 lanes of each warp's quarter of tensor memory.
 template <int HN, int KB>
 __global__ void __launch_bounds__(kDecodeThreads, 1)
 latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmC, const __grid_constant__ CUtensorMap tmR, DecodeParams p) {
   constexpr int kQPanel = HN * 128;  // bytes of a 64-column panel of HN rows
-  constexpr int kKeyPanel = KB * 128, kPairBytes = 2 * kKeyPanel;
+  constexpr int kKeyPanel = KB * 128, kPairBytes = 2 * kKeyPanel, kPBytes = KB / 64 * kQPanel;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   uint8_t* sC = smem;                                        // [ring] pieces: KB rows x 128 columns
   uint8_t* sR = sC + p.ring * kPairBytes;                    // [rot_stages]
   uint8_t* sQ = sR + p.rot_stages * p.rot_panels * kKeyPanel;  // 2 * pairs latent panels, then the rotated ones
-  uint8_t* sP = sQ + (2 * p.pairs + p.rot_panels) * kQPanel;     // [HN heads, KB keys]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + KB / 64 * kQPanel);
+  uint8_t* sP = sQ + (2 * p.pairs + p.rot_panels) * kQPanel;     // [2] tiles of [HN heads, KB keys]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kPBytes);
   uint64_t* c_full = bars;                 // [ring]
   uint64_t* c_empty = bars + kMaxRing;     // [ring]
   uint64_t* r_full = bars + 2 * kMaxRing;  // [rot_stages <= 2]
@@ -472,9 +472,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   uint64_t* s_full = r_empty + 2;          // [2]
   uint64_t* s_free = s_full + 2;           // [2]
   uint64_t* q_full = s_free + 2;
-  uint64_t* p_full = q_full + 1;           // reused alternately with pv_done below
-  uint64_t* pv_done = p_full + 1;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 1);
+  uint64_t* p_full = q_full + 1;           // [2]
+  uint64_t* pv_done = p_full + 2;          // [2]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(pv_done + 2);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
   float* s_red = reinterpret_cast<float*>(tmem_slot + 2);  // [4][HN]
 
@@ -499,10 +499,10 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       mbar_init(&r_empty[i], 1);
       mbar_init(&s_full[i], 1);
       mbar_init(&s_free[i], 4);
+      mbar_init(&p_full[i], 4);
+      mbar_init(&pv_done[i], 1);
     }
     mbar_init(q_full, 1);
-    mbar_init(p_full, 4);
-    mbar_init(pv_done, 1);
     *abort_flag = 0;
     fence_mbar_init();
   }
@@ -514,8 +514,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
-  const uint32_t tS[2] = {tmem_base, tmem_base + HN};
-  const uint32_t tO = tmem_base + 2 * HN;
+  const uint32_t tO = tmem_base + 2 * HN;  // after the two score tiles
 
   if (warp == 0) {
     // ---------------------------------------------------------------- TMA producer
@@ -553,67 +552,73 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       if (++rs == p.rot_stages) rs = 0, rph ^= 1;
     }
   } else if (warp == 1) {
-    // ---------------------------------------------------------------- MMA issuer
-    constexpr uint32_t idesc_s = make_idesc_bf16(128, HN, false, false);
-    constexpr uint32_t idesc_o = make_idesc_bf16(128, HN, true, false);
-    const uint32_t aC = smem_u32(sC), aR = smem_u32(sR), aQ = smem_u32(sQ), aP = smem_u32(sP);
-    const uint64_t dC = make_smem_desc_sw128(aC, 16, 1024), dR = make_smem_desc_sw128(aR, 16, 1024), dQ = make_smem_desc_sw128(aQ, 16, 1024);
-    const uint64_t dCt = make_smem_desc_sw128(aC, kKeyPanel, 1024), dP = make_smem_desc_sw128(aP, 16, 1024);
-    auto issue_s = [&](int it) -> bool {
-      const int st = it & 1, rs = it % p.rot_stages;
-      if (!mbar_wait(&s_free[st], ((it >> 1) & 1) ^ 1)) return false;
-      for (int u = 0; u < p.pairs; ++u) {
-        const int n = it * p.pairs + u, slot = n % p.ring;
-        if (!mbar_wait(&c_full[slot], (n / p.ring) & 1)) return false;
+    // ---------------------------------------------------------------- scores: Sᵀ(it) = C(it) · Qᵀ
+    // With few columns an MMA is over in less time than its issue takes, so scores and outputs are issued by two warps.
+    constexpr uint32_t idesc = make_idesc_bf16(KB, HN, false, false);
+    const uint64_t dC = make_smem_desc_sw128(smem_u32(sC), 16, 1024), dR = make_smem_desc_sw128(smem_u32(sR), 16, 1024), dQ = make_smem_desc_sw128(smem_u32(sQ), 16, 1024);
+    bool ok = n_blocks == 0 || mbar_wait(q_full, 0);
+    int cs = 0, rs = 0;
+    uint32_t cph = 0, rph = 0;
+    for (int it = 0; it < n_blocks && ok && !*abort_flag; ++it) {
+      const int st = it & 1;
+      const uint32_t tS = tmem_base + st * HN;
+      ok = mbar_wait(&s_free[st], ((it >> 1) & 1) ^ 1);
+      for (int u = 0; u < p.pairs && ok; ++u) {
+        ok = mbar_wait(&c_full[cs], cph);
         tc_fence_after();
-        if (lane == 0) {
-          const uint64_t da = dC + slot * (kPairBytes >> 4), db = dQ + u * (2 * kQPanel >> 4);
+        if (ok && elect_one()) {
+          const uint64_t da = dC + cs * (kPairBytes >> 4), db = dQ + u * (2 * kQPanel >> 4);
           const int steps = p.c_steps - 8 * u;
-          umma_panel(tS[st], da, db, steps, idesc_s, u > 0);
-          umma_panel(tS[st], da + (kKeyPanel >> 4), db + (kQPanel >> 4), steps - 4, idesc_s, true);
+          umma_panel(tS, da, db, steps, idesc, u > 0);
+          umma_panel(tS, da + (kKeyPanel >> 4), db + (kQPanel >> 4), steps - 4, idesc, true);
         }
         __syncwarp();
+        if (++cs == p.ring) cs = 0, cph ^= 1;
       }
-      if (!mbar_wait(&r_full[rs], (it / p.rot_stages) & 1)) return false;
+      ok = ok && mbar_wait(&r_full[rs], rph);
       tc_fence_after();
-      if (lane == 0) {
+      if (ok && elect_one()) {
         for (int j = 0; j < p.rot_panels; ++j)
-          umma_panel(tS[st], dR + (rs * p.rot_panels + j) * (kKeyPanel >> 4), dQ + (2 * p.pairs + j) * (kQPanel >> 4), p.rot_steps - 4 * j, idesc_s, true);
+          umma_panel(tS, dR + (rs * p.rot_panels + j) * (kKeyPanel >> 4), dQ + (2 * p.pairs + j) * (kQPanel >> 4), p.rot_steps - 4 * j, idesc, true);
         umma_commit(&r_empty[rs]);
         umma_commit(&s_full[st]);
       }
       __syncwarp();
-      return true;
-    };
-    bool ok = n_blocks == 0 || mbar_wait(q_full, 0);
-    if (ok && n_blocks > 0) ok = issue_s(0);
-    for (int it = 0; it < n_blocks && ok && !*abort_flag; ++it) {
-      if (p.lookahead && it + 1 < n_blocks) ok = issue_s(it + 1);
-      if (!ok || !mbar_wait(p_full, it & 1)) {
-        ok = false;
-        break;
-      }
-      tc_fence_after();
-      if (lane == 0) {
-        for (int u = 0; u < p.pairs; ++u) {
-          const int slot = (it * p.pairs + u) % p.ring;
-          const uint64_t da = dCt + slot * (kPairBytes >> 4);
-#pragma unroll
-          for (int k = 0; k < KB / 16; ++k)
-            umma_f16(tO + u * HN, da + k * (2048 >> 4), dP + (k >> 2) * (kQPanel >> 4) + (k & 3) * 2, idesc_o, (it | k) != 0);
-          umma_commit(&c_empty[slot]);
-        }
-        umma_commit(pv_done);
-      }
-      __syncwarp();
-      if (!p.lookahead && it + 1 < n_blocks) ok = issue_s(it + 1);
+      if (++rs == p.rot_stages) rs = 0, rph ^= 1;
     }
     if (!ok) fail(abort_flag, p.err, 232);
+  } else if (warp == 3) {
+    // ---------------------------------------------------------------- outputs: Oᵀ += C(it)ᵀ · Pᵀ(it), then the pieces are handed back
+    constexpr uint32_t idesc = make_idesc_bf16(128, HN, true, false);
+    const uint64_t dC = make_smem_desc_sw128(smem_u32(sC), kKeyPanel, 1024), dP = make_smem_desc_sw128(smem_u32(sP), 16, 1024);
+    bool ok = true;
+    int cs = 0;
+    uint32_t cph = 0;
+    for (int it = 0; it < n_blocks && ok && !*abort_flag; ++it) {
+      ok = mbar_wait(&p_full[it & 1], (it >> 1) & 1);
+      const uint64_t db = dP + (it & 1) * (kPBytes >> 4);
+      for (int u = 0; u < p.pairs && ok; ++u) {
+        ok = mbar_wait(&c_full[cs], cph);
+        tc_fence_after();
+        if (ok && elect_one()) {
+          const uint64_t da = dC + cs * (kPairBytes >> 4);
+#pragma unroll
+          for (int k = 0; k < KB / 16; ++k) umma_f16(tO + u * HN, da + k * (2048 >> 4), db + (k >> 2) * (kQPanel >> 4) + (k & 3) * 2, idesc, (it | k) != 0);
+          umma_commit(&c_empty[cs]);
+          if (u + 1 == p.pairs) umma_commit(&pv_done[it & 1]);
+        }
+        __syncwarp();
+        if (++cs == p.ring) cs = 0, cph ^= 1;
+      }
+    }
+    if (!ok) fail(abort_flag, p.err, 234);
   } else if (warp >= 4) {
     // ---------------------------------------------------------------- softmax over the keys of a tile: one key per thread, all heads
     // After a failed wait the warp keeps going without waiting, so all four warps meet at the same named barriers.
     const int quarter = warp & 3;
     const int r = quarter * 32 + lane;
+    const int r_key = KB == 64 ? quarter * 16 + lane : r;  // this thread's key of a tile ...
+    const bool has_key = KB == 128 || lane < 16;           // ... if it has one
     const uint32_t lane_sel = static_cast<uint32_t>(quarter * 32) << 16;
     const float c = p.scale * kLog2e;
     float m[HN], l[HN];
@@ -622,16 +627,16 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     bool ok = true;
     for (int it = 0; it < n_blocks; ++it) {
       const int st = it & 1;
-      const int key = (first + it) * KB + r;
+      const int key = (first + it) * KB + r_key;
       if (ok && !*abort_flag) ok = mbar_wait(&s_full[st], (it >> 1) & 1);
       tc_fence_after();
       uint32_t sv[HN];
-      tmem_ld_heads<HN>(tS[st] + lane_sel, sv);
+      tmem_ld_heads<HN>(tmem_base + st * HN + lane_sel, sv);
       tmem_ld_wait();
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(&s_free[st]);
-      const bool visible = r < KB && key >= lo && key <= hi;
+      const bool visible = has_key && key >= lo && key <= hi;
       bool grows = false;
 #pragma unroll
       for (int h = 0; h < HN; ++h) {
@@ -663,25 +668,26 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         l[h] += e;
         sv[h] = __float_as_uint(e);
       }
-      if (it > 0) {  // the previous outputs are finished: P may be overwritten and O rescaled
-        if (ok && !*abort_flag) ok = mbar_wait(pv_done, (it - 1) & 1);
+      // P(it) may be overwritten once the outputs of tile it - 2 are finished; the running outputs may be rescaled only once those of
+      // tile it - 1 are (a maximum rarely moves after the first tiles)
+      if (it > 1 && ok && !*abort_flag) ok = mbar_wait(&pv_done[it & 1], ((it >> 1) & 1) ^ 1);
+      if (it > 0 && update) {
+        if (ok && !*abort_flag) ok = mbar_wait(&pv_done[(it - 1) & 1], ((it - 1) >> 1) & 1);
         tc_fence_after();
-        if (update) {
 #pragma unroll 1
-          for (int u = 0; u < p.pairs; ++u) {
-            uint32_t v[HN];
-            tmem_ld_heads<HN>(tO + lane_sel + u * HN, v);
-            tmem_ld_wait();
+        for (int u = 0; u < p.pairs; ++u) {
+          uint32_t v[HN];
+          tmem_ld_heads<HN>(tO + lane_sel + u * HN, v);
+          tmem_ld_wait();
 #pragma unroll
-            for (int h = 0; h < HN; ++h) v[h] = __float_as_uint(__uint_as_float(v[h]) * alpha[h]);
-            tmem_st_heads<HN>(tO + lane_sel + u * HN, v);
-          }
-          tmem_st_wait();
+          for (int h = 0; h < HN; ++h) v[h] = __float_as_uint(__uint_as_float(v[h]) * alpha[h]);
+          tmem_st_heads<HN>(tO + lane_sel + u * HN, v);
         }
+        tmem_st_wait();
       }
-      if (r < KB) {
-        uint8_t* panel = sP + (r >> 6) * kQPanel;
-        const int chunk = (r & 63) >> 3, byte = (r & 7) * 2;
+      if (has_key) {
+        uint8_t* panel = sP + (it & 1) * kPBytes + (r_key >> 6) * kQPanel;
+        const int chunk = (r_key & 63) >> 3, byte = (r_key & 7) * 2;
 #pragma unroll
         for (int h = 0; h < HN; ++h)
           *reinterpret_cast<__nv_bfloat16*>(panel + h * 128 + ((chunk ^ (h & 7)) << 4) + byte) = __float2bfloat16_rn(__uint_as_float(sv[h]));
@@ -689,9 +695,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       fence_proxy_async_smem();
       tc_fence_before();
       __syncwarp();
-      if (lane == 0) mbar_arrive(p_full);
+      if (lane == 0) mbar_arrive(&p_full[it & 1]);
     }
-    if (ok && n_blocks > 0 && !*abort_flag) ok = mbar_wait(pv_done, (n_blocks - 1) & 1);
+    if (ok && n_blocks > 0 && !*abort_flag) ok = mbar_wait(&pv_done[(n_blocks - 1) & 1], ((n_blocks - 1) >> 1) & 1);
     if (!ok) fail(abort_flag, p.err, 233);
     tc_fence_after();
     group_sync();  // the last maxima have been read
@@ -740,7 +746,7 @@ static int map3(CUtensorMap* m, const void* base, uint64_t d0, uint64_t d1, uint
 template <int HN, int KB>
 static int plan_decode(DecodeParams& p) {
   const int q_panel = HN * 128, key_panel = KB * 128;
-  const int fixed = (2 * p.pairs + p.rot_panels + KB / 64) * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
+  const int fixed = (2 * p.pairs + p.rot_panels + 2 * (KB / 64)) * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
   const int rot_bytes = p.rot_panels * key_panel;
   p.rot_stages = fixed + 2 * rot_bytes + 2 * p.pairs * 2 * key_panel <= kSmemLimit ? 2 : 1;
   int ring = (kSmemLimit - fixed - p.rot_stages * rot_bytes) / (2 * key_panel);

@@ -248,6 +248,7 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
   const T* wp = w + static_cast<long long>(h) * K * N + n;
   if (n < N)  // the weights are on their way while the rows are staged
     for (int k = warp; k < K; k += 8) asm volatile("prefetch.global.L2 [%0];" ::"l"(wp + static_cast<long long>(k) * N));
+#pragma unroll 4
   for (int t = threadIdx.x; t < kRows * K; t += 256) {
     const int r = t / K, k = t - r * K;
     sA[t] = r0 + r < R ? to_f(a[(r0 + r) * a_row + static_cast<long long>(h) * a_head + k]) : 0.f;
@@ -352,19 +353,21 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const float* __restri
     if (n0 + c < N)
       for (int k = lane * (128 / static_cast<int>(sizeof(T))); k < K; k += 32 * (128 / static_cast<int>(sizeof(T))))
         asm volatile("prefetch.global.L2 [%0];" ::"l"(wp + static_cast<long long>(c) * K + k));
-  for (int t = threadIdx.x; t < ROWS * K; t += 256) {
-    const int r = t / K, k = t - r * K;
-    float v = 0.f;
-    if (r0 + r < R) {
-      const long long rh = static_cast<long long>(r0 + r) * heads + h;
-      float inv = 1.f;
-      if (ml != nullptr) {
-        const float l = ml[rh].y;
-        inv = l > 0.f ? 1.f / l : 0.f;
-      }
-      v = inv == 0.f ? 0.f : o[rh * K + k] * inv;
-    }
-    sA[t] = v;
+  const int vec_k = K / VEC;
+#pragma unroll 4
+  for (int t = threadIdx.x; t < ROWS * vec_k; t += 256) {
+    const int r = t / vec_k, k = (t - r * vec_k) * VEC;
+    float f[VEC];
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) f[v] = 0.f;
+    if (r0 + r < R) WVec<float, VEC>::load(o + (static_cast<long long>(r0 + r) * heads + h) * K + k, f);
+#pragma unroll
+    for (int v = 0; v < VEC; ++v) sA[r * K + k + v] = f[v];
+  }
+  float inv = 1.f;  // of row `lane`
+  if (ml != nullptr && lane < ROWS && r0 + lane < R) {
+    const float l = ml[static_cast<long long>(r0 + lane) * heads + h].y;
+    inv = l > 0.f ? 1.f / l : 0.f;
   }
   __syncthreads();
 #pragma unroll
@@ -391,7 +394,7 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const float* __restri
       acc[r] = warp_sum(acc[r]);
       if (lane == r && r0 + r < R) {
         const long long col = static_cast<long long>(h) * N + n;
-        float v = acc[r];
+        float v = inv == 0.f ? 0.f : acc[r] * inv;  // a row without keys was never written
         if (gate != nullptr) v *= sigmoid_as<T>(to_f(gate[(r0 + r) * gate_ld + col]));
         out[static_cast<long long>(r0 + r) * heads * N + col] = from_f<T>(v);
       }
