@@ -212,10 +212,10 @@ def test_decode_and_value(shape, kind, vdim, monkeypatch):
             out = latent.value(o, ml, w, g, vdim=vdim)
             _errors()
             _close(out, want, dtype)
-        monkeypatch.setattr(latent, "GROUPED_ROWS", 1)
+        monkeypatch.setattr(latent, "VALUE_GROUPED_ROWS", 1)
         if dtype == BF16:
             _close(latent.value(o, ml, w, g, vdim=vdim), want, dtype)
-        monkeypatch.setattr(latent, "GROUPED_ROWS", 32)
+        monkeypatch.setattr(latent, "VALUE_GROUPED_ROWS", 32)
 
 
 def test_decode_single_key_stands_out():
@@ -242,7 +242,7 @@ def test_decode_single_key_stands_out():
 
 
 @pytest.mark.parametrize("dtype", [BF16, F32])
-@pytest.mark.parametrize("rows", [1, 3, 9, 40])
+@pytest.mark.parametrize("rows", [1, 3, 9, 130])
 @pytest.mark.parametrize("heads,dim,rot,rank", [(3, 24, 8, 48), (16, 128, 64, 512), (5, 12, 6, 10)])
 def test_absorb(dtype, rows, heads, dim, rot, rank):
     from torchtune_b200.ops import latent
@@ -250,7 +250,7 @@ def test_absorb(dtype, rows, heads, dim, rot, rank):
     q = _rand(rows, heads * (dim + rot) + 8, dtype=dtype, seed=1)[:, : heads * (dim + rot)]
     w = _rand(heads * dim, rank, dtype=dtype, seed=2, scale=dim**-0.5)
     out = torch.zeros(rows, heads, rank + rot, dtype=dtype, device=DEV)
-    latent.absorb(q.contiguous() if rows == 40 else q, w, out, heads=heads, dim=dim, rot=rot, rank=rank)
+    latent.absorb(q.contiguous() if rows == 130 else q, w, out, heads=heads, dim=dim, rot=rot, rank=rank)
     want = np.einsum("rhd,hdn->rhn", _np(q).reshape(rows, heads, dim + rot)[..., :dim], _np(w).reshape(heads, dim, rank))
     _errors()
     _close(out[..., :rank], want, dtype, tol16=1e-2)

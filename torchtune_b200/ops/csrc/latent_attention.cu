@@ -166,7 +166,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       if (++vs == p.v_stages) vs = 0, vph ^= 1;
     }
   } else if (warp == 1) {
-    // ---------------------------------------------------------------- MMA issuer
+    // ---------------------------------------------------------------- MMA issuer (an elected lane: the compiler then keeps descriptors uniform)
     constexpr uint32_t idesc_s = make_idesc_bf16(128, 128, false, false);
     const uint32_t idesc_o = make_idesc_bf16(128, p.v_panels * 64, false, true);
     const uint32_t aQ = smem_u32(sQ), aK = smem_u32(sK), aV = smem_u32(sV);
@@ -180,7 +180,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
         k_ready = j;
       }
       tc_fence_after();
-      if (lane == 0) {
+      if (elect_one()) {
         const uint32_t q_base = aQ + x * q_bytes, k_base = aK + st * q_bytes;
         for (int k = 0; k < p.dim_steps; ++k) umma_f16(tS[x], desc_kmajor(q_base, k), desc_kmajor(k_base, k), idesc_s, k != 0);
         const uint32_t off = p.dim_panels * kPanelBytes;
@@ -211,7 +211,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
           v_ready = j;
         }
         tc_fence_after();
-        if (lane == 0) {
+        if (elect_one()) {
           const uint64_t dv = desc_mnmajor(aV + st * v_bytes, 0);
 #pragma unroll
           for (int k = 0; k < kBlk / 16; ++k) umma_f16_ts(tO[x], tS[x] + k * 8, dv + k * (2048 >> 4), idesc_o, (n | k) != 0);

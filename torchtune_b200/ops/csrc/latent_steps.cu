@@ -297,14 +297,18 @@ __device__ __forceinline__ float warp_max_of(float v) {
   return v;
 }
 
+static constexpr int kCombineGroups = 4;  // groups of 128 threads, each adding up every fourth range
+
 template <bool HEAD_MAJOR>
-__global__ void __launch_bounds__(128) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits, int R,
-                                                             int heads, int K) {
+__global__ void __launch_bounds__(128 * kCombineGroups) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits,
+                                                                              int R, int heads, int K) {
   extern __shared__ float wts[];  // [splits]: exp2(m_s - m) / sum, 0 for a split without keys (which has written nothing)
-  const int r = blockIdx.x, h = blockIdx.y;
+  __shared__ float part[kCombineGroups][128];
+  const int r = blockIdx.x, h = blockIdx.y, group = threadIdx.x >> 7, col = threadIdx.x & 127;
   const long long rh = static_cast<long long>(r) * heads + h, RH = static_cast<long long>(R) * heads;
   if (threadIdx.x < 32) {
     float m = -INFINITY, l = 0.f;
+#pragma unroll 2
     for (int s = threadIdx.x; s < splits; s += 32) {
       const float2 v = ml[s * RH + rh];
       if (v.y > 0.f) {
@@ -322,15 +326,21 @@ __global__ void __launch_bounds__(128) latent_combine_kernel(const float* __rest
     }
   }
   __syncthreads();
-  const int k = blockIdx.z * 128 + threadIdx.x;
+  const int k = blockIdx.z * 128 + col;
+  float acc = 0.f;
   if (k < K) {
-    float acc = 0.f;
     const float* src = o + rh * K + k;
-#pragma unroll 16
-    for (int s = 0; s < splits; ++s) {
+#pragma unroll 8
+    for (int s = group; s < splits; s += kCombineGroups) {
       const float v = src[s * RH * K];  // loaded in any case, so the loads of many ranges are in flight together
       acc += wts[s] != 0.f ? wts[s] * v : 0.f;
     }
+  }
+  part[group][col] = acc;
+  __syncthreads();
+  if (group == 0 && k < K) {
+#pragma unroll
+    for (int g = 1; g < kCombineGroups; ++g) acc += part[g][col];
     if constexpr (HEAD_MAJOR) static_cast<__nv_bfloat16*>(out)[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(acc);
     else static_cast<float*>(out)[rh * K + k] = acc;
   }
@@ -370,31 +380,35 @@ __global__ void __launch_bounds__(256) latent_value_kernel(const float* __restri
     inv = l > 0.f ? 1.f / l : 0.f;
   }
   __syncthreads();
+  if (n0 >= N) return;
+  const bool two = n0 + 1 < N;  // the two columns of a warp share every read of the rows
+  float acc[2][ROWS];
 #pragma unroll
-  for (int c = 0; c < 2; ++c) {
-    const int n = n0 + c;
-    if (n >= N) break;
-    float acc[ROWS];
-#pragma unroll
-    for (int r = 0; r < ROWS; ++r) acc[r] = 0.f;
+  for (int r = 0; r < ROWS; ++r) acc[0][r] = acc[1][r] = 0.f;
 #pragma unroll 4
-    for (int k = lane * VEC; k < K; k += 32 * VEC) {
-      float f[VEC];
-      WVec<T, VEC>::load(wp + static_cast<long long>(c) * K + k, f);
-#pragma unroll
-      for (int r = 0; r < ROWS; ++r) {
-        float a[VEC];
-        WVec<float, VEC>::load_shared(sA + r * K + k, a);
-#pragma unroll
-        for (int v = 0; v < VEC; ++v) acc[r] += a[v] * f[v];
-      }
-    }
+  for (int k = lane * VEC; k < K; k += 32 * VEC) {
+    float f[VEC], g[VEC];
+    WVec<T, VEC>::load(wp + k, f);
+    WVec<T, VEC>::load(wp + (two ? K : 0) + k, g);
 #pragma unroll
     for (int r = 0; r < ROWS; ++r) {
-      acc[r] = warp_sum(acc[r]);
-      if (lane == r && r0 + r < R) {
-        const long long col = static_cast<long long>(h) * N + n;
-        float v = inv == 0.f ? 0.f : acc[r] * inv;  // a row without keys was never written
+      float a[VEC];
+      WVec<float, VEC>::load_shared(sA + r * K + k, a);
+#pragma unroll
+      for (int v = 0; v < VEC; ++v) {
+        acc[0][r] += a[v] * f[v];
+        acc[1][r] += a[v] * g[v];
+      }
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < 2; ++c) {
+#pragma unroll
+    for (int r = 0; r < ROWS; ++r) {
+      const float sum = warp_sum(acc[c][r]);
+      if (lane == r && r0 + r < R && (c == 0 || two)) {
+        const long long col = static_cast<long long>(h) * N + n0 + c;
+        float v = inv == 0.f ? 0.f : sum * inv;  // a row without keys was never written
         if (gate != nullptr) v *= sigmoid_as<T>(to_f(gate[(r0 + r) * gate_ld + col]));
         out[static_cast<long long>(r0 + r) * heads * N + col] = from_f<T>(v);
       }
@@ -656,8 +670,8 @@ extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, in
   auto st = static_cast<cudaStream_t>(stream);
   auto m = reinterpret_cast<const float2*>(ml);
   TTB_COUNT_LAUNCH(1);
-  if (head_major) latent_combine_kernel<true><<<dim3(rows, heads, (K + 127) / 128), 128, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
-  else latent_combine_kernel<false><<<dim3(rows, heads, (K + 127) / 128), 128, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
+  if (head_major) latent_combine_kernel<true><<<dim3(rows, heads, (K + 127) / 128), 128 * kCombineGroups, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
+  else latent_combine_kernel<false><<<dim3(rows, heads, (K + 127) / 128), 128 * kCombineGroups, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 

@@ -13,7 +13,9 @@ import torch
 from ._lib import check, err_word, lib, stream_ptr
 
 _SMS = None
-GROUPED_ROWS = 32  # from this many decoded rows the per-head products run as grouped tensor-core GEMMs
+# from this many decoded rows the per-head products run as grouped tensor-core GEMMs
+ABSORB_GROUPED_ROWS = 128
+VALUE_GROUPED_ROWS = 32
 
 
 @dataclass
@@ -105,7 +107,7 @@ def absorb(q: torch.Tensor, w_uk: torch.Tensor, q_lat: torch.Tensor, *, heads: i
     """``q_lat[:, h, :rank] = W_uk[h]ᵀ q_n[h]`` for ``q`` ``[rows, heads·(dim+rot)]``."""
     rows = q.shape[0]
     assert w_uk.shape == (heads * dim, rank) and w_uk.is_contiguous() and w_uk.dtype == q.dtype and q_lat.shape == (rows, heads, rank + rot)
-    if q.dtype == torch.bfloat16 and rows >= GROUPED_ROWS and dim % 8 == 0 and rank % 8 == 0:
+    if q.dtype == torch.bfloat16 and rows >= ABSORB_GROUPED_ROWS and dim % 8 == 0 and rank % 8 == 0:
         from ._cuda import _grouped_gemm
 
         a = q.view(rows, heads, dim + rot)[:, :, :dim].transpose(0, 1).reshape(heads * rows, dim)
@@ -156,7 +158,7 @@ def value(o: torch.Tensor, ml: torch.Tensor, w_uv: torch.Tensor, gate: Optional[
     assert w_uv.shape == (heads * vdim, rank) and w_uv.is_contiguous() and (gate is None or gate.shape == (rows, heads * vdim))
     out = torch.empty(rows, heads * vdim, dtype=w_uv.dtype, device=o.device)
     gate_ld = 0 if gate is None else _pitch(gate)
-    if w_uv.dtype == torch.bfloat16 and rows >= GROUPED_ROWS and vdim % 8 == 0 and rank % 8 == 0:
+    if w_uv.dtype == torch.bfloat16 and rows >= VALUE_GROUPED_ROWS and vdim % 8 == 0 and rank % 8 == 0:
         from ._cuda import _grouped_gemm
 
         lat = torch.empty(heads * rows, rank, dtype=torch.bfloat16, device=o.device)
