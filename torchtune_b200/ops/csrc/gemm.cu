@@ -394,7 +394,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA_ptr, const CUte
           __syncwarp();
         }
         tc_fence_after();
-        if (lane == 0) {
+        if (elect_one()) {  // an elected lane rather than lane 0: descriptors stay uniform and an MMA's issue takes half the time
           const uint32_t sa = smem_u32(smem + stage * Cfg::kStageBytes);
           const uint32_t sb = sa + Cfg::kABytes;
 #pragma unroll
@@ -420,7 +420,7 @@ __device__ __forceinline__ void gemm_body(const CUtensorMap* tmA_ptr, const CUte
         if (lane == 0) atomicExch(p.err, 103);
         break;
       }
-      if (lane == 0) umma_commit(&tfull[acc]);
+      if (elect_one()) umma_commit(&tfull[acc]);
       __syncwarp();
       if (++acc == 2) {
         acc = 0;
