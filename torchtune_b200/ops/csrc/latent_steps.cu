@@ -297,13 +297,12 @@ __device__ __forceinline__ float warp_max_of(float v) {
   return v;
 }
 
-static constexpr int kCombineGroups = 4;  // groups of 128 threads, each adding up every fourth range
-
-template <bool HEAD_MAJOR>
-__global__ void __launch_bounds__(128 * kCombineGroups) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits,
+// GROUPS groups of 128 threads, each adding up every GROUPS-th range: several when there are many ranges (few rows).
+template <bool HEAD_MAJOR, int GROUPS>
+__global__ void __launch_bounds__(128 * GROUPS) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits,
                                                                               int R, int heads, int K) {
   extern __shared__ float wts[];  // [splits]: exp2(m_s - m) / sum, 0 for a split without keys (which has written nothing)
-  __shared__ float part[kCombineGroups][128];
+  __shared__ float part[GROUPS][128];
   const int r = blockIdx.x, h = blockIdx.y, group = threadIdx.x >> 7, col = threadIdx.x & 127;
   const long long rh = static_cast<long long>(r) * heads + h, RH = static_cast<long long>(R) * heads;
   if (threadIdx.x < 32) {
@@ -331,16 +330,18 @@ __global__ void __launch_bounds__(128 * kCombineGroups) latent_combine_kernel(co
   if (k < K) {
     const float* src = o + rh * K + k;
 #pragma unroll 8
-    for (int s = group; s < splits; s += kCombineGroups) {
+    for (int s = group; s < splits; s += GROUPS) {
       const float v = src[s * RH * K];  // loaded in any case, so the loads of many ranges are in flight together
       acc += wts[s] != 0.f ? wts[s] * v : 0.f;
     }
   }
-  part[group][col] = acc;
-  __syncthreads();
+  if constexpr (GROUPS > 1) {
+    part[group][col] = acc;
+    __syncthreads();
+  }
   if (group == 0 && k < K) {
 #pragma unroll
-    for (int g = 1; g < kCombineGroups; ++g) acc += part[g][col];
+    for (int g = 1; g < GROUPS; ++g) acc += part[g][col];
     if constexpr (HEAD_MAJOR) static_cast<__nv_bfloat16*>(out)[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(acc);
     else static_cast<float*>(out)[rh * K + k] = acc;
   }
@@ -670,8 +671,16 @@ extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, in
   auto st = static_cast<cudaStream_t>(stream);
   auto m = reinterpret_cast<const float2*>(ml);
   TTB_COUNT_LAUNCH(1);
-  if (head_major) latent_combine_kernel<true><<<dim3(rows, heads, (K + 127) / 128), 128 * kCombineGroups, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
-  else latent_combine_kernel<false><<<dim3(rows, heads, (K + 127) / 128), 128 * kCombineGroups, splits * 4, st>>>(o, m, out, splits, rows, heads, K);
+  const dim3 grid(rows, heads, (K + 127) / 128);
+#define TTB_COMBINE(HEAD_MAJOR, GROUPS) latent_combine_kernel<HEAD_MAJOR, GROUPS><<<grid, 128 * GROUPS, splits * 4, st>>>(o, m, out, splits, rows, heads, K)
+  if (splits < 8) {
+    if (head_major) TTB_COMBINE(true, 1);
+    else TTB_COMBINE(false, 1);
+  } else {
+    if (head_major) TTB_COMBINE(true, 4);
+    else TTB_COMBINE(false, 4);
+  }
+#undef TTB_COMBINE
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 
