@@ -70,9 +70,13 @@ class DecodeGraph:
         mask = layout.mask(used, 1)
 
         def body() -> torch.Tensor:
-            for c in self.caches:
-                c.rewind(used)
             return hidden_states(model, self.tokens, input_pos=(self.slot - self.start).clamp_min_(0)[:, None], mask=mask)
+
+        saved = [c.snapshot() for c in self.caches]  # the first launches are a step of their own, undone before the recording
+
+        def undo() -> None:
+            for c, before in zip(self.caches, saved):
+                c.restore(before)
 
         for c in self.caches:
             c.slot = self.slot
@@ -82,6 +86,7 @@ class DecodeGraph:
             with torch.cuda.stream(side):  # first launches and their one-time set-up stay out of the recording
                 body()
             torch.cuda.current_stream(dev).wait_stream(side)
+            undo()
             self.graph = torch.cuda.CUDAGraph()
             with torch.cuda.graph(self.graph):
                 self.hidden = body()
@@ -89,7 +94,7 @@ class DecodeGraph:
         finally:
             for c in self.caches:
                 c.slot = None
-                c.rewind(used)
+            undo()
         self._next = used
 
     def __call__(self, tokens: torch.Tensor) -> torch.Tensor:

@@ -11,15 +11,18 @@ adapter description and produces the same module tree / state-dict keys
 from __future__ import annotations
 
 from dataclasses import dataclass, field
-from typing import Callable, List, Optional, Sequence
+from typing import Callable, List, Optional, Sequence, Tuple
 
 import torch
 from torch import nn
 
 from ..modules import (
+    CachedMixer,
     FeedForward,
     FrozenNF4Linear,
+    HyperConnectionLayer,
     LatentAttention,
+    LayerScale,
     Linear,
     MultiHeadAttention,
     ResidualStreamLayer,
@@ -99,6 +102,11 @@ class DecoderArch:
     residual_stream: bool = False
     residual_mult: float = 1.0
     wide_logits: bool = False
+    # several 32-bit residual streams with layer scales (0: one stream); learned position embeddings (table length, 0: none); a run of
+    # layers (start, stop, times) that is repeated
+    streams: int = 0
+    learned_positions: int = 0
+    loop: Optional[Tuple[int, int, int]] = None
 
     def resolved_head_dim(self) -> int:
         return self.head_dim or self.embed_dim // self.num_heads
@@ -181,6 +189,11 @@ def build_decoder(arch: DecoderArch, adapter: Optional[AdapterSpec] = None) -> T
             layers.append(ResidualStreamLayer(attn, mlp, sa_norm=norm(), sa_scale=norm(), mlp_norm=norm() if mlp is not None else None,
                                               mlp_scale=norm() if mlp is not None else None, residual_mult=arch.residual_mult))
             continue
+        if arch.streams:
+            norm = lambda: arch.norm(arch.embed_dim, arch.norm_eps)  # noqa: E731
+            layers.append(HyperConnectionLayer(attn, mlp, streams=arch.streams, sa_norm=norm(), sa_scale=LayerScale(arch.embed_dim), mlp_norm=norm() if mlp is not None else None,
+                                               mlp_scale=LayerScale(arch.embed_dim) if mlp is not None else None))
+            continue
         layers.append(
             TransformerSelfAttentionLayer(
                 attn=attn,
@@ -214,7 +227,11 @@ def build_decoder(arch: DecoderArch, adapter: Optional[AdapterSpec] = None) -> T
     )
     model.logit_softcap = float(arch.logit_softcap)
     model.wide_logits = bool(arch.wide_logits)
-    model.span_masks = all(isinstance(layer.attn, LatentAttention) for layer in layers)
+    model.span_masks = all(isinstance(layer.attn, (LatentAttention, CachedMixer)) for layer in layers)
+    if arch.learned_positions:
+        model.pos_embeddings = nn.Embedding(arch.learned_positions, arch.embed_dim)
+    if arch.loop is not None:
+        model.set_loop(*arch.loop)
     if ad.quantize_base:
         # checkpoints of a quantised-base model are written in bf16 on CPU
         _register_reparametrize_state_dict_hooks(model, dtype=tok.weight.dtype)

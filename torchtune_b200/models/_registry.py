@@ -9,7 +9,7 @@ import json
 import tempfile
 from dataclasses import dataclass
 from pathlib import Path
-from typing import Any, Dict, Optional, Union
+from typing import Any, Dict, Mapping, Optional, Union
 
 import torch
 from torch import nn
@@ -23,11 +23,24 @@ class Architecture:
 
 ARCHITECTURES: Dict[str, Architecture] = {
     "Begapel": Architecture("torchtune_b200.models.begapel.begapel", "BEGAPEL"),
+    "Ragenex": Architecture("torchtune_b200.models.ragenex.ragenex", "RAGENEX"),
 }
 
 
 def read_config(folder: Union[str, Path]) -> Dict[str, Any]:
-    return json.loads((Path(folder) / "config.json").read_text())
+    return as_mapping(Path(folder) / "config.json")
+
+
+def as_mapping(config: Union[str, Path, Mapping[str, Any]]) -> Dict[str, Any]:
+    """A model configuration given as a mapping, a ``config.json`` or the folder that holds one."""
+    if isinstance(config, (str, Path)):
+        path = Path(config)
+        return json.loads((path / "config.json" if path.is_dir() else path).read_text())
+    if hasattr(config, "to_dict"):
+        return config.to_dict()
+    from ..config import DictConfig, OmegaConf
+
+    return OmegaConf.to_container(config) if isinstance(config, DictConfig) else dict(config)
 
 
 def architecture_of(config: Dict[str, Any]) -> Architecture:

@@ -1,8 +1,6 @@
 """``begapel(config)`` / ``lora_begapel(..., config=...)`` from a ``config.json`` (a mapping or the path of the file)."""
 from __future__ import annotations
 
-import json
-from pathlib import Path
 from typing import Any, Dict, List, Mapping, Tuple, Union
 
 from torch import nn
@@ -11,20 +9,10 @@ from ...modules import LatentAttention, RMSNorm, StreamRMSNorm
 from ...modules.latent_attention import PreciseRotaryPositionalEmbeddings
 from .._factory import AdapterSpec, DecoderArch, build_mlp
 from .._generic import component_builders
+from .._registry import as_mapping
 
 _MIXER = "latent_attention"
 _ATTN_MODULES = {"q_proj", "kv_down", "k_up", "v_up", "gate_proj", "output_proj"}
-
-
-def _read(config: Union[str, Path, Mapping[str, Any]]) -> Dict[str, Any]:
-    if isinstance(config, (str, Path)):
-        path = Path(config)
-        return json.loads((path / "config.json" if path.is_dir() else path).read_text())
-    if hasattr(config, "to_dict"):
-        return config.to_dict()
-    from ...config import DictConfig, OmegaConf
-
-    return OmegaConf.to_container(config) if isinstance(config, DictConfig) else dict(config)
 
 
 def _check_layers(layers: List[Dict[str, Any]]) -> None:
@@ -51,7 +39,7 @@ def _check_layers(layers: List[Dict[str, Any]]) -> None:
 
 
 def _arch(config: Union[str, Mapping[str, Any]], max_seq_len: int = 32768) -> DecoderArch:
-    cfg = _read(config)
+    cfg = as_mapping(config)
     layers, dim, eps = cfg["layers"], int(cfg["width"]), float(cfg["norm"]["eps"])
     _check_layers(layers)
     ropes: Dict[Tuple[int, float], nn.Module] = {}

@@ -9,11 +9,14 @@ from .common_utils import (
     slice_str_to_array,
 )
 from .embedding_utils import resize_token_embeddings
-from .feed_forward import FeedForward
-from .kv_cache import KVCache
+from .cached_mixer import CachedMixer
+from .feed_forward import ClampedGLU, FeedForward
+from .hyper_connections import HyperConnection, LayerScale
+from .kv_cache import KVCache, PassCaches, RowCache, SpanKVCache, StateCache
 from .latent_attention import LatentAttention, LatentCache
 from .layer_norm import Fp32LayerNorm
 from .linear import Linear
+from .linear_attention import LightningAttention
 from .low_precision import FrozenNF4Linear
 from .position_embeddings import (
     HalfSplitRotaryPositionalEmbeddings,
@@ -24,10 +27,11 @@ from .position_embeddings import (
     RotaryPositionalEmbeddings,
     VisionRotaryPositionalEmbeddings,
 )
-from .rms_norm import RMSNorm, StreamRMSNorm, rms_norm
+from .rms_norm import RMSNorm, StreamLayerNorm, StreamRMSNorm, rms_norm
+from .span_attention import QueryTemperature, SpanAttention
 from .tanh_gate import TanhGate
 from .tied_linear import TiedLinear
-from .transformer import ResidualStreamLayer, TransformerCrossAttentionLayer, TransformerDecoder, TransformerSelfAttentionLayer
+from .transformer import HyperConnectionLayer, ResidualStreamLayer, TransformerCrossAttentionLayer, TransformerDecoder, TransformerSelfAttentionLayer
 from .layer_dropout import LayerDropout, ModuleLayerDropoutWrapper, ScaleType, get_scale, prepare_layer_dropout
 from .vq_embeddings import VectorQuantizedEmbeddings
 from .vision_transformer import CLSEmbedding, CLSProjection, PatchEmbedding, VisionTransformer
@@ -47,11 +51,17 @@ __all__ = [
     "CLSProjection",
     "PatchEmbedding",
     "TanhGate",
+    "CachedMixer",
+    "ClampedGLU",
     "FeedForward",
     "FrozenNF4Linear",
+    "HyperConnection",
+    "HyperConnectionLayer",
     "KVCache",
     "LatentAttention",
     "LatentCache",
+    "LayerScale",
+    "LightningAttention",
     "Linear",
     "RotaryPositionalEmbeddings",
     "VisionRotaryPositionalEmbeddings",
@@ -60,7 +70,14 @@ __all__ = [
     "HalfSplitRotaryPositionalEmbeddings",
     "Qwen2RotaryPositionalEmbeddings",
     "Phi3RotaryPositionalEmbeddings",
+    "PassCaches",
+    "QueryTemperature",
     "RMSNorm",
+    "RowCache",
+    "SpanAttention",
+    "SpanKVCache",
+    "StateCache",
+    "StreamLayerNorm",
     "StreamRMSNorm",
     "rms_norm",
     "TiedLinear",

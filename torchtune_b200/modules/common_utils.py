@@ -58,9 +58,10 @@ def slice_str_to_array(slice_str: str, length: int) -> List[bool]:
 
 def _attention_modules(model: nn.Module):
     from .attention import MultiHeadAttention
+    from .cached_mixer import CachedMixer
     from .latent_attention import LatentAttention
 
-    return [m for m in model.modules() if isinstance(m, (MultiHeadAttention, LatentAttention))]
+    return [m for m in model.modules() if isinstance(m, (MultiHeadAttention, LatentAttention, CachedMixer))]
 
 
 @contextlib.contextmanager

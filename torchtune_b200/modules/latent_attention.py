@@ -21,7 +21,8 @@ from torch import nn
 
 from .. import ops
 from ..ops import reference
-from ..ops.mask import AttentionMask
+from ._spans import dense, dense_visibility, join, joined, kernel_bounds, plain, positions
+from .kv_cache import RowCache
 from .position_embeddings import RotaryPositionalEmbeddings
 
 logger = logging.getLogger(__name__)
@@ -41,48 +42,15 @@ class PreciseRotaryPositionalEmbeddings(RotaryPositionalEmbeddings):
         self.is_cache_built = True
 
 
-class LatentCache(nn.Module):
-    """Latent rows ``[batch, max_seq_len, width]`` of the tokens seen so far; all batch rows append at the same slot.
-
-    ``slot`` is ``None`` (the next slot is known to the host) or a device int32 that holds it, so a captured decode step can be replayed."""
+class LatentCache(RowCache):
+    """Latent rows ``[batch, max_seq_len, width]`` of the tokens seen so far."""
 
     def __init__(self, batch_size: int, max_seq_len: int, width: int, dtype: torch.dtype) -> None:
-        super().__init__()
+        super().__init__(batch_size, max_seq_len)
         self.register_buffer("latent", torch.zeros(batch_size, max_seq_len, width, dtype=dtype), persistent=False)
-        self.batch_size = batch_size
-        self.max_seq_len = max_seq_len
-        self.slot: Optional[torch.Tensor] = None
-        self._size = 0
 
-    @property
-    def size(self) -> int:
-        return self._size
-
-    def reset(self) -> None:
-        self._size = 0
-
-    def reserve(self, batch: int, count: int) -> int:
-        """Slot of the first of ``count`` new tokens."""
-        if batch > self.latent.shape[0]:
-            raise ValueError(f"The current cache has been setup with a batch size of {self.latent.shape[0]}, but found new tokens with batch size {batch}!")
-        if self._size + count > self.max_seq_len:
-            raise AssertionError("KV cache is full: cannot write past max_seq_len")
-        return self._size
-
-    def advance(self, count: int) -> None:
-        self._size += count
-
-    def rewind(self, size: int) -> None:
-        """Forgets the tokens from slot ``size`` on."""
-        if not 0 <= size <= self.max_seq_len:
-            raise ValueError(f"{size} is outside the cache")
-        self._size = size
-
-    def keep_rows(self, rows: List[int]) -> None:
-        """Drops every batch row that is not in ``rows`` (increasing) and moves the kept ones to the front."""
-        for to, row in enumerate(rows):
-            if to != row:
-                self.latent[to, : self._size].copy_(self.latent[row, : self._size])
+    def _move_row(self, row: int, to: int) -> None:
+        self.latent[to, : self._size].copy_(self.latent[row, : self._size])
 
 
 class LatentAttention(nn.Module):
@@ -145,24 +113,10 @@ class LatentAttention(nn.Module):
     def _inputs(self) -> List[nn.Module]:
         return [m for m in (self.q_proj, self.kv_down, self.gate_proj) if m is not None]
 
-    @staticmethod
-    def _join(mods: List[nn.Module]) -> None:
-        """Lays the weights of plain linears that read the same input out as one matrix (the parameters become views of it), so
-        inference multiplies them in one GEMM."""
-        weights = [m.weight for m in mods] if all(_plain(m) for m in mods) else []
-        if len(weights) < 2 or any(w.device.type == "meta" or hasattr(w, "_grad_buffer") for w in weights) or _joined(mods) is not None:
-            return
-        whole = torch.cat([w.data for w in weights])
-        at = 0
-        for w in weights:
-            n = w.shape[0]
-            w.data = whole[at : at + n]
-            at += n
-
     def _join_projections(self) -> None:
         with torch.no_grad():
-            self._join(self._inputs())
-            self._join([self.k_up, self.v_up])
+            join(self._inputs())
+            join([self.k_up, self.v_up])
 
     # ------------------------------------------------------------------ forward
     def forward(self, x: torch.Tensor, y: Optional[torch.Tensor] = None, *, mask=None, input_pos: Optional[torch.Tensor] = None,
@@ -176,7 +130,7 @@ class LatentAttention(nn.Module):
             raise RuntimeError(f"layer {self.layer_index} reads the latents of layer {self.latent_from}, which has not run in this pass")
         if ops.cuda_ops_enabled(x) and x.dtype in (torch.bfloat16, torch.float32):
             if not (torch.is_grad_enabled() and (x.requires_grad or any(p.requires_grad for p in self.parameters()))):
-                bounds = _kernel_bounds(state, mask, x, self._first_slot(state))
+                bounds = kernel_bounds(state, mask, x, self._first_slot(state))
                 if bounds is not None:
                     return self._forward_kernels(x, bounds, input_pos, state)
                 ops._fallback("latent_attention", "a mask whose rows are not key ranges", x)
@@ -192,7 +146,7 @@ class LatentAttention(nn.Module):
     def _project(self, x2: torch.Tensor) -> Tuple[torch.Tensor, Optional[torch.Tensor], Optional[torch.Tensor]]:
         """Queries, latent input and gate as 2-D tensors with contiguous rows."""
         mods = self._inputs()
-        whole = _joined(mods)
+        whole = joined(mods)
         if whole is not None:
             parts = ops.linear(x2, whole).split([m.weight.shape[0] for m in mods], dim=1)
         else:
@@ -206,7 +160,7 @@ class LatentAttention(nn.Module):
         b, s, _ = x.shape
         H, d, r, dv, rank = self.num_heads, self.head_dim, self.rot_dim, self.value_dim, self.kv_rank
         q, kv, gate = self._project(x.reshape(b * s, -1))
-        pos = _positions(state, input_pos, b, s)
+        pos = positions(state, input_pos, b, s)
         if self.latent_from is None:
             cache = self.kv_cache if self.cache_enabled else None
             if cache is not None:
@@ -228,14 +182,14 @@ class LatentAttention(nn.Module):
             if cache is not None:
                 cache.advance(s)
         if decode:
-            latent.absorb(q, self.k_up.weight if _plain(self.k_up) else _dense(self.k_up), q_lat, heads=H, dim=d, rot=r, rank=rank)
+            latent.absorb(q, self.k_up.weight if plain(self.k_up) else dense(self.k_up), q_lat, heads=H, dim=d, rot=r, rank=rank)
             keys = first + 1 if slot is None else buf.shape[1]
             o, ml = latent.decode(q_lat, buf, rank=rank, rot=r, scale=self.scale, slot=slot, slot_host=first, bounds=bounds, keys=keys)
-            out = latent.value(o, ml, self.v_up.weight if _plain(self.v_up) else _dense(self.v_up), gate, vdim=dv)
+            out = latent.value(o, ml, self.v_up.weight if plain(self.v_up) else dense(self.v_up), gate, vdim=dv)
         else:
             sk = first + s
             lat = buf[:, :sk, :rank].reshape(b * sk, rank)
-            whole = _joined([self.k_up, self.v_up])
+            whole = joined([self.k_up, self.v_up])
             if whole is not None:
                 kn, v = ops.linear(lat, whole).split([H * d, H * dv], dim=1)
             else:
@@ -269,95 +223,8 @@ class LatentAttention(nn.Module):
             rows, first, _, cache = state["latent", self.latent_from]
         sk = first + s
         lat, k_rot = rows[:, :sk, :rank], rows[:, :sk, rank:]
-        visible = _dense_visibility(mask, b, s, sk, first, x.device)
+        visible = dense_visibility(mask, b, s, sk, first, x.device)
         out = reference.latent_attention(q, self.k_up(lat).view(b, sk, H, d), k_rot, self.v_up(lat).view(b, sk, H, dv), visible, self.scale).reshape(b, s, H * dv)
         if self.gate_proj is not None:
             out = (out.float() * torch.sigmoid(self.gate_proj(x).float())).to(out.dtype)
         return self.output_proj(out)
-
-
-def _plain(m: Optional[nn.Module]) -> bool:
-    return isinstance(m, nn.Linear) and type(m).__name__ == "Linear" and m.bias is None
-
-
-def _dense(m: nn.Module) -> torch.Tensor:
-    """The matrix an adapted or quantised linear stands for (``[out, in]``)."""
-    eye = torch.eye(m.in_dim if hasattr(m, "in_dim") else m.in_features, dtype=next(m.parameters()).dtype, device=next(m.parameters()).device)
-    return m(eye).t().contiguous()
-
-
-def _joined(mods: List[nn.Module]) -> Optional[torch.Tensor]:
-    """The one matrix the weights of ``mods`` are consecutive row blocks of, or ``None``."""
-    if len(mods) < 2 or not all(_plain(m) for m in mods):
-        return None
-    w0 = mods[0].weight.data
-    at, store = w0.data_ptr(), w0.untyped_storage().data_ptr()
-    rows = 0
-    for m in mods:
-        w = m.weight.data
-        if not w.is_contiguous() or w.data_ptr() != at or w.untyped_storage().data_ptr() != store or w.shape[1] != w0.shape[1]:
-            return None
-        at += w.numel() * w.element_size()
-        rows += w.shape[0]
-    return torch.as_strided(w0, (rows, w0.shape[1]), (w0.shape[1], 1))
-
-
-def _positions(state: Dict[Any, Any], input_pos: Optional[torch.Tensor], b: int, s: int) -> Optional[torch.Tensor]:
-    if input_pos is None:
-        return None
-    key = ("positions", input_pos.data_ptr(), tuple(input_pos.shape))
-    if key not in state:
-        state[key] = (input_pos.reshape(-1, s).expand(b, s).to(torch.int32).contiguous(), input_pos)
-    return state[key][0]
-
-
-def _kernel_bounds(state: Dict[Any, Any], mask, x: torch.Tensor, first: int):
-    """Key range of every query for the kernels, once per pass; ``None`` for a boolean mask that is not a set of growing ranges."""
-    key = ("bounds", first, id(mask))
-    if key not in state:
-        state[key] = (_make_bounds(mask, x.shape[0], x.shape[1], first, x.device), mask)
-    return state[key][0]
-
-
-def _make_bounds(mask, b: int, s: int, first: int, device):
-    from ..ops._cuda_attention import dense_mask_bounds, lower_bounds
-    from ..ops.latent import Bounds
-
-    if mask is None:
-        return Bounds()
-    if isinstance(mask, AttentionMask) and mask.bool_mask is None:
-        if mask.key_start is not None:
-            if mask.key_start.numel() != b:
-                raise ValueError(f"key_start has {mask.key_start.numel()} rows, the batch has {b}")
-            return Bounds(lo=mask.key_start.to(device=device, dtype=torch.int32).contiguous(), lo_row=1)
-        if not mask.causal:
-            return None
-        lo = lower_bounds(mask, b, s, device)
-        if lo is None:
-            return Bounds()
-        return Bounds(lo=lo.contiguous(), lo_row=s, lo_query=1) if first == 0 else None
-    dense = mask.bool_mask if isinstance(mask, AttentionMask) else mask
-    dense = dense[..., : first + s]
-    if dense.dim() == 4 and dense.shape[1] != 1:
-        return None
-    bits, lo, hi = dense_mask_bounds(dense, b, s, first + s)
-    empty = hi < lo
-    ranges = bits.sum(-1, dtype=torch.int32) == torch.where(empty, 0, hi - lo + 1)
-    growing = ((lo[:, 1:] >= lo[:, :-1]) & (hi[:, 1:] >= hi[:, :-1])).all() if s > 1 else torch.tensor(True, device=device)
-    if not bool(ranges.all() & growing):
-        return None
-    return Bounds(lo=lo, lo_row=s, lo_query=1, hi=hi, hi_row=s, hi_query=1)
-
-
-def _dense_visibility(mask, b: int, s: int, sk: int, first: int, device) -> torch.Tensor:
-    if isinstance(mask, AttentionMask):
-        if mask.bool_mask is None and mask.key_start is None and s != sk:
-            if mask.doc_ids is not None or mask.chunk > 0 or mask.window > 0:
-                raise ValueError("document, chunk and window masks need the whole sequence in one pass")
-        else:
-            m = mask.dense(b, s, sk, device)
-            mask = torch.ones(1, s, sk, dtype=torch.bool, device=device) if m is None else m
-    if mask is None or isinstance(mask, AttentionMask):
-        return (torch.arange(sk, device=device)[None, :] <= first + torch.arange(s, device=device)[:, None]).unsqueeze(0)
-    m = mask[:, 0] if mask.dim() == 4 else mask
-    return m[..., :sk]

@@ -54,6 +54,22 @@ class StreamRMSNorm(nn.Module):
         return f"dim={self.normalized_shape[0]}, eps={self.eps}, offset={self.offset}"
 
 
+class StreamLayerNorm(nn.Module):
+    """Layer norm with a gain and no bias between a 32-bit residual stream and a sublayer: fp32 in, the gain's dtype out, one rounding."""
+
+    def __init__(self, dim: int, eps: float = 1e-5) -> None:
+        super().__init__()
+        self.normalized_shape = (dim,)
+        self.eps = eps
+        self.scale = nn.Parameter(torch.ones(dim))
+
+    def forward(self, x: torch.Tensor) -> torch.Tensor:
+        return ops.stream_step(x.float().unsqueeze(-2), None, None, None, None, None, self.scale, eps=self.eps, centered=True)[1]
+
+    def extra_repr(self) -> str:
+        return f"dim={self.normalized_shape[0]}, eps={self.eps}"
+
+
 def rms_norm(x: torch.Tensor, eps: float = 1e-6) -> torch.Tensor:
     """Weight-less RMS norm over the last dimension (Llama-4 q/k normalisation)."""
     return ops.rms_norm(x, None, eps)

@@ -2,7 +2,7 @@
 from __future__ import annotations
 
 import copy
-from typing import Callable, List, Optional, Union
+from typing import Callable, List, Optional, Tuple, Union
 
 import torch
 from torch import nn
@@ -10,7 +10,9 @@ from torch import nn
 from .. import ops
 from ..ops.mask import AttentionMask
 from .attention import MaskLike, MultiHeadAttention
-from .rms_norm import StreamRMSNorm
+from .cached_mixer import CachedMixer
+from .hyper_connections import HyperConnection, LayerScale, StreamEntry
+from .rms_norm import StreamLayerNorm, StreamRMSNorm
 
 
 class TransformerSelfAttentionLayer(nn.Module):
@@ -106,6 +108,42 @@ class ResidualStreamLayer(TransformerSelfAttentionLayer):
         return x if next_norm is None else (x, normed)
 
 
+class HyperConnectionLayer(TransformerSelfAttentionLayer):
+    """Pre-norm decoder layer on several 32-bit residual streams (:class:`~torchtune_b200.modules.HyperConnection`) with layer scales; the
+    feed-forward block is left out with ``mlp=None``.
+
+    The end of one sublayer and the norm in front of the next run as one pass over the streams.  A decoder that chains layers passes
+    ``(streams, normed input)`` and the :class:`~torchtune_b200.modules.hyper_connections.StreamEntry` of what follows this layer, and
+    receives the same kind of pair for it.  A plain ``[b, s, dim]`` input stands for streams that are all equal."""
+
+    def __init__(self, attn: nn.Module, mlp: Optional[nn.Module], *, streams: int, sa_norm: StreamLayerNorm, sa_scale: LayerScale, mlp_norm: Optional[StreamLayerNorm] = None,
+                 mlp_scale: Optional[LayerScale] = None) -> None:
+        nn.Module.__init__(self)
+        if (mlp is None) != (mlp_norm is None) or (mlp is None) != (mlp_scale is None):
+            raise ValueError("the feed-forward block, its norm and its scale come together")
+        self.attn, self.mlp = attn, mlp
+        self.sa_norm, self.sa_scale, self.mlp_norm, self.mlp_scale = sa_norm, sa_scale, mlp_norm, mlp_scale
+        self.sa_streams = HyperConnection(streams)
+        self.mlp_streams = HyperConnection(streams) if mlp is not None else None
+        self.mask_mod = None
+
+    @property
+    def entry(self) -> StreamEntry:
+        return StreamEntry(self.sa_streams.read, self.sa_norm)
+
+    def forward(self, x, *, mask: MaskLike = None, input_pos: Optional[torch.Tensor] = None, layer_state: Optional[dict] = None, following: Optional[StreamEntry] = None, **kwargs):
+        x, normed = x if isinstance(x, tuple) else (x, None)
+        if x.dim() == 3:
+            x = x.float().unsqueeze(2)
+        if normed is None:
+            normed = HyperConnection.enter(x, self.entry)
+        y = self.attn(normed, mask=mask, input_pos=input_pos, layer_state=layer_state)
+        x, normed = self.sa_streams.step(x, y, self.sa_scale, following if self.mlp is None else StreamEntry(self.mlp_streams.read, self.mlp_norm))
+        if self.mlp is not None:
+            x, normed = self.mlp_streams.step(x, self.mlp(normed), self.mlp_scale, following)
+        return x if following is None else (x, normed)
+
+
 class TransformerCrossAttentionLayer(nn.Module):
     """Cross-attention block over encoder tokens.  Query rows whose encoder mask is
     empty contribute nothing (attention and MLP outputs are zeroed for them)."""
@@ -178,6 +216,12 @@ class TransformerCrossAttentionLayer(nn.Module):
         return h + self.mlp_scale(mlp_out)
 
 
+def _collapsed(h) -> torch.Tensor:
+    """The hidden state a layer leaves: the sum of its streams where it has several."""
+    h = h[0] if isinstance(h, tuple) else h
+    return h.sum(2) if h.dim() == 4 else h
+
+
 def _get_clones(module: nn.Module, n: int) -> nn.ModuleList:
     return nn.ModuleList([copy.deepcopy(module) for _ in range(n)])
 
@@ -233,8 +277,32 @@ class TransformerDecoder(nn.Module):
         self.wide_logits = False
         # Prompts of unequal length may be described to the layers by the first key of every row instead of a boolean mask.
         self.span_masks = False
+        # Learned embeddings of the positions, added to the token embeddings (fp32 sum).
+        self.pos_embeddings: Optional[nn.Embedding] = None
+        # Layers ``start … stop - 1`` run ``times`` times in a row before the rest follows.
+        self.loop: Optional[Tuple[int, int, int]] = None
         self.encoder_max_cache_seq_len = None
         self.decoder_max_cache_seq_len = None
+
+    # -- order of the layers ---------------------------------------------------
+    def set_loop(self, start: int, stop: int, times: int) -> None:
+        """Runs the layers ``start … stop - 1`` ``times`` times in a row, each time with a cache of its own."""
+        if not 0 <= start < stop <= len(self.layers) or times < 1:
+            raise ValueError(f"layers {start} … {stop} cannot run {times} times in a decoder of {len(self.layers)} layers")
+        if self.caches_are_setup():
+            raise RuntimeError("the order of the layers is fixed once caches exist")
+        for layer in self.layers[start:stop]:
+            if times > 1 and not isinstance(layer.attn, CachedMixer):
+                raise ValueError(f"{type(layer.attn).__name__} keeps one cache and cannot run several times")
+            layer.attn.num_passes = times
+        self.loop = (start, stop, times)
+
+    def run_order(self) -> List[Tuple[int, int]]:
+        """``(layer, pass)`` in the order of execution."""
+        start, stop, times = self.loop or (0, 0, 0)
+        order = [(i, 0) for i in range(start)]
+        order += [(i, n) for n in range(times) for i in range(start, stop)]
+        return order + [(i, 0) for i in range(stop, len(self.layers))]
 
     # -- output chunking (deprecated path kept for API parity) -------------
     def set_num_output_chunks(self, num_output_chunks: int) -> None:
@@ -309,21 +377,28 @@ class TransformerDecoder(nn.Module):
             raise ValueError("Exactly one of `tokens` or `input_embeds` must be provided.")
         seq_len = tokens.shape[1] if input_embeds is None else input_embeds.shape[1]
         self._validate_inputs(seq_len, mask=mask, encoder_input=encoder_input, encoder_mask=encoder_mask, input_pos=input_pos)
-        h = ops.embed_tokens(self.tok_embeddings, tokens) if input_embeds is None else input_embeds
+        h = self._embed(tokens, input_embeds, input_pos)
         hidden = []
         layer_state: dict = {}
-        kinds = [getattr(layer, "inner_cls", type(layer)) for layer in self.layers]
-        for i, layer in enumerate(self.layers):
+        order = self.run_order()
+        for i, (idx, run) in enumerate(order):
+            layer = self.layers[idx]
             if i in self.output_hidden_states:
-                hidden.append(h[0] if isinstance(h, tuple) else h)
+                hidden.append(_collapsed(h))
             extra = {}
-            if kinds[i] is ResidualStreamLayer:
-                following = getattr(self.layers[i + 1], "sa_norm", None) if i + 1 < len(self.layers) else self.norm
+            kind = getattr(layer, "inner_cls", type(layer))
+            after = self.layers[order[i + 1][0]] if i + 1 < len(order) else None
+            if kind is ResidualStreamLayer:
+                following = getattr(after, "sa_norm", None) if after is not None else self.norm
                 extra = {"layer_state": layer_state, "next_norm": following if isinstance(following, StreamRMSNorm) else None}
+            elif kind is HyperConnectionLayer:
+                layer_state["pass"] = run
+                last = StreamEntry(None, self.norm, keep=len(order) in self.output_hidden_states)
+                extra = {"layer_state": layer_state, "following": last if after is None else after.entry}
             h = layer(h, mask=mask, encoder_input=encoder_input, encoder_mask=encoder_mask, input_pos=input_pos, **extra)
+        if len(order) in self.output_hidden_states:
+            hidden.append(_collapsed(h))
         h, normed = h if isinstance(h, tuple) else (h, None)
-        if len(self.layers) in self.output_hidden_states:
-            hidden.append(h)
         h = self.norm(h) if normed is None else normed
         if self.skip_output_layer:
             output = h
@@ -332,6 +407,16 @@ class TransformerDecoder(nn.Module):
         else:
             output = self.unembed_normed(h)
         return output if not hidden else [*hidden, output]
+
+    def _embed(self, tokens: Optional[torch.Tensor], input_embeds: Optional[torch.Tensor], input_pos: Optional[torch.Tensor]) -> torch.Tensor:
+        if self.pos_embeddings is None:
+            return ops.embed_tokens(self.tok_embeddings, tokens) if input_embeds is None else input_embeds
+        b, s = (tokens if input_embeds is None else input_embeds).shape[:2]
+        pos = torch.arange(s, device=self.pos_embeddings.weight.device) if input_pos is None else input_pos
+        pos = pos.reshape(-1, s).expand(b, s)
+        if input_embeds is not None:
+            return input_embeds.float() + self.pos_embeddings(pos).float()
+        return ops.embed_positions(tokens, pos, self.tok_embeddings.weight, self.pos_embeddings.weight)
 
     def unembed_normed(self, h: torch.Tensor) -> torch.Tensor:
         if self.wide_logits and type(self.output).__name__ == "Linear" and self.output.bias is None:

@@ -32,6 +32,9 @@ __all__ = [
     "linear_residual",
     "linear_wide",
     "residual_norm",
+    "stream_step",
+    "embed_positions",
+    "clamped_glu",
     "softcap",
     "rms_norm",
     "rope",
@@ -240,6 +243,44 @@ def residual_norm(x: torch.Tensor, y: Optional[torch.Tensor], w_post: Optional[t
 
         return latent.residual_norm(x, y, w_post, w_next, eps, mult, offset)
     return reference.residual_norm(x, y, w_post, w_next, eps=eps, mult=mult, offset=offset)
+
+
+def stream_step(x: torch.Tensor, y: Optional[torch.Tensor], gain: Optional[torch.Tensor], mix: Optional[torch.Tensor], out: Optional[torch.Tensor], read: Optional[torch.Tensor],
+                w_next: Optional[torch.Tensor], *, eps: float, centered: bool, offset: float = 0.0, keep: bool = True) -> Tuple[Optional[torch.Tensor], Optional[torch.Tensor]]:
+    """The step between two sublayers on several 32-bit residual streams ``x`` ``[..., S, D]`` (one stream stands for S equal ones):
+    ``x'_t = Σ_s mix[s, t] x_s + out[t] · gain · y`` (``y=None``: ``x' = x``) and ``h = norm(Σ_t read[t] x'_t)`` in the gain's dtype (``read=None``: ones;
+    ``w_next=None``: no ``h``), where norm is a layer norm without bias (``centered``) or an RMS norm times ``offset + w_next``, all in fp32.
+    Returns ``(x', h)``; ``keep=False`` says that ``x'`` is not needed."""
+    w = w_next if w_next is not None else gain
+    grads = torch.is_grad_enabled() and any(t is not None and t.requires_grad for t in (x, y, gain, mix, out, read, w_next))
+    if cuda_ops_enabled(x) and x.dtype == torch.float32 and not grads and w.dtype in (torch.bfloat16, torch.float32) and (y is None or y.dtype == w.dtype) and x.numel() > 0:
+        from . import streams
+
+        return streams.stream_step(x, y, gain, mix, out, read, w_next, eps, centered, offset, keep)
+    lead = x.shape[:-2]
+    x4 = x.reshape(1, -1, *x.shape[-2:])
+    x4, h = reference.stream_step(x4, None if y is None else y.reshape(1, -1, y.shape[-1]), gain, mix, out, read, w_next, eps=eps, centered=centered, offset=offset)
+    return x4.view(*lead, *x4.shape[-2:]), None if h is None else h.view(*lead, h.shape[-1])
+
+
+def embed_positions(tokens: torch.Tensor, positions: torch.Tensor, table: torch.Tensor, pos_table: torch.Tensor) -> torch.Tensor:
+    """``table[tokens] + pos_table[positions]`` summed in fp32, ``[b, s, D]``."""
+    grads = torch.is_grad_enabled() and (table.requires_grad or pos_table.requires_grad)
+    if cuda_ops_enabled(table) and not grads and table.dtype == pos_table.dtype and table.dtype in (torch.bfloat16, torch.float32) and tokens.numel() > 0:
+        from . import streams
+
+        return streams.embed_positions(tokens, positions, table, pos_table)
+    return F.embedding(tokens, table).float() + F.embedding(positions.long(), pos_table).float()
+
+
+def clamped_glu(gate: torch.Tensor, up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """``g · sigmoid(alpha · g) · (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``."""
+    grads = torch.is_grad_enabled() and (gate.requires_grad or up.requires_grad)
+    if _native(gate, (torch.bfloat16, torch.float32)) and up.dtype == gate.dtype and not grads and gate.numel() > 0:
+        from . import streams
+
+        return streams.clamped_glu(gate, up, limit, alpha)
+    return reference.clamped_glu(gate, up, limit, alpha)
 
 
 def rope(

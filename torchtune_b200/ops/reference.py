@@ -8,7 +8,7 @@ restates.
 from __future__ import annotations
 
 import math
-from typing import Optional, Tuple
+from typing import Optional, Sequence, Tuple
 
 import torch
 import torch.nn.functional as F
@@ -45,6 +45,77 @@ def latent_attention(q: torch.Tensor, k_up: torch.Tensor, k_rot: torch.Tensor, v
     s = (torch.einsum("bqhd,bkhd->bhqk", qf[..., :d], k_up.float()) + torch.einsum("bqhr,bkr->bhqk", qf[..., d:], k_rot.float())) * scale
     p = torch.nan_to_num(torch.softmax(s.masked_fill(~visible.unsqueeze(1), float("-inf")), dim=-1), nan=0.0)
     return torch.einsum("bhqk,bkhd->bqhd", p, v.float()).to(q.dtype)
+
+
+def span_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, visible: torch.Tensor, scale: float) -> torch.Tensor:
+    """Grouped-query attention with separate key and value sizes: ``q`` ``[b, s, h, d]``, ``k`` ``[b, sk, g, d]``, ``v`` ``[b, sk, g, dv]``,
+    ``visible`` ``[b | 1, s, sk]``.  Scores and weights in fp32; a row without keys gives 0."""
+    b, s, h, d = q.shape
+    g = k.shape[2]
+    sc = torch.einsum("bqgnd,bkgd->bgnqk", q.float().view(b, s, g, h // g, d), k.float()) * scale
+    p = torch.nan_to_num(torch.softmax(sc.masked_fill(~visible[:, None, None], float("-inf")), dim=-1), nan=0.0)
+    return torch.einsum("bgnqk,bkgd->bqgnd", p, v.float()).reshape(b, s, h, -1).to(q.dtype)
+
+
+def decay_powers(decay: Sequence[float], count: int) -> torch.Tensor:
+    """``decay ** (0 … count - 1)`` per head, evaluated in double precision (0 ** 0 = 1)."""
+    return torch.tensor(decay, dtype=torch.float64)[:, None] ** torch.arange(count, dtype=torch.float64)[None, :]
+
+
+def lightning_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: Sequence[float], state: Optional[torch.Tensor], chunk: int = 128) -> Tuple[torch.Tensor, torch.Tensor]:
+    """``S_t = λ S_{t-1} + k_t v_tᵀ``, ``o_t = S_tᵀ q_t`` per head, chunk by chunk in fp32: ``q`` / ``k`` ``[b, s, h, d]``, ``v`` ``[b, s, h, dv]``, ``state``
+    ``[b, h, d, dv]`` (``None``: zeros).  Returns ``(o [b, s, h, dv], state)``, both fp32."""
+    b, s, h, d = q.shape
+    q, k, v = (t.float().transpose(1, 2) for t in (q, k, v))
+    state = torch.zeros(b, h, d, v.shape[-1], device=q.device) if state is None else state.float()
+    pw = decay_powers(decay, chunk + 1).float().to(q.device)
+    out = []
+    for c0 in range(0, s, chunk):
+        qc, kc, vc = (t[:, :, c0 : c0 + chunk] for t in (q, k, v))
+        n = qc.shape[2]
+        age = torch.arange(n, device=q.device)[:, None] - torch.arange(n, device=q.device)[None, :]
+        w = torch.where(age >= 0, pw[:, age.clamp_min(0)], 0.0)
+        inside = (qc @ kc.transpose(-1, -2) * w) @ vc
+        out.append(inside + pw[:, 1 : n + 1, None] * (qc @ state))
+        state = pw[:, n, None, None] * state + (kc * pw[:, :n].flip(1)[..., None]).transpose(-1, -2) @ vc
+    return torch.cat(out, dim=2).transpose(1, 2), state
+
+
+def gated_norm(o: torch.Tensor, gain: torch.Tensor, gate: torch.Tensor, eps: float) -> torch.Tensor:
+    """``o / rms(o) · gain · sigmoid(gate)`` in fp32, in the gain's dtype."""
+    of = o.float()
+    y = of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps) * gain.float()
+    return (y * torch.sigmoid(gate.float())).to(gain.dtype)
+
+
+def clamped_glu(gate: torch.Tensor, up: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """``g · sigmoid(alpha · g) · (u + 1)`` with ``g = min(gate, limit)`` and ``u = clamp(up, -limit, limit)``."""
+    g, u = gate.float().clamp(max=limit), up.float().clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1.0)).to(gate.dtype)
+
+
+def stream_norm(x: torch.Tensor, w: torch.Tensor, eps: float, centered: bool, offset: float) -> torch.Tensor:
+    """Layer norm without bias (``centered``) or RMS norm of ``x`` in fp32, times ``offset + w``, in the gain's dtype."""
+    xf = x.float()
+    if centered:
+        xf = xf - xf.mean(-1, keepdim=True)
+    return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * (offset + w.float())).to(w.dtype)
+
+
+def stream_step(x: torch.Tensor, y: Optional[torch.Tensor], gain: Optional[torch.Tensor], mix: Optional[torch.Tensor], out: Optional[torch.Tensor], read: Optional[torch.Tensor],
+                w_next: Optional[torch.Tensor], *, eps: float, centered: bool, offset: float = 0.0) -> Tuple[torch.Tensor, Optional[torch.Tensor]]:
+    """Residual streams ``x`` ``[b, s, S | 1, D]`` fp32 (one stream stands for S equal ones): ``x'_t = Σ_s mix[s, t] x_s + out[t] · gain · y`` (``y=None``: ``x' = x``),
+    ``h = norm(Σ_t read[t] x'_t; w_next)`` (``read=None``: ones; ``w_next=None``: no ``h``)."""
+    if y is not None:
+        S = mix.shape[0]
+        x = torch.einsum("bnsd,st->bntd", x.expand(-1, -1, S, -1), mix.float()) + out.float()[:, None] * (gain.float() * y.float())[:, :, None]
+    if w_next is None:
+        return x, None
+    if read is None:
+        u = x.sum(2)
+    else:
+        u = (x.expand(-1, -1, read.numel(), -1) * read.float()[:, None]).sum(2)
+    return x, stream_norm(u, w_next, eps, centered, offset)
 
 
 def rope_interleaved(x: torch.Tensor, cache: torch.Tensor, input_pos: Optional[torch.Tensor]) -> torch.Tensor:

@@ -58,6 +58,7 @@ def _load_family_codecs() -> None:
         "phi3._convert_weights",
         "qwen2._convert_weights",
         "qwen3._convert_weights",
+        "ragenex._convert_weights",
         "gemma2._convert_weights",
         "llama4._convert_weights",
         "llama3_2_vision._convert_weights",

@@ -67,6 +67,7 @@ class ModelType(Enum):
     PHI4 = "phi4"
     REWARD = "reward"
     QWEN2 = "qwen2"
+    RAGENEX = "ragenex"
     CLIP_TEXT = "clip_text"
     T5_ENCODER = "t5_encoder"
     QWEN3 = "qwen3"
