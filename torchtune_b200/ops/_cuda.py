@@ -1089,10 +1089,11 @@ class _GateUpSwiGLU(torch.autograd.Function):
     """``silu(x · W1ᵀ) ⊙ (x · W3ᵀ)`` as one launch of the CTA-pair GEMM: the even CTA of a pair loads rows of ``W1``, the odd one the same
     rows of ``W3``, and the epilogue applies the activation (``csrc/gemm2sm.cu``, SWIGLU form).  In a gradient-free pass (the first forward
     under activation checkpointing) the two pre-activations never reach HBM; otherwise the epilogue also stores them for backward, which
-    is the existing SwiGLU-backward kernel followed by the usual input- and weight-gradient GEMMs."""
+    is the existing SwiGLU-backward kernel followed by the usual input- and weight-gradient GEMMs.  ``clamp`` ``(limit, alpha)`` selects the
+    clamped gate instead (no backward)."""
 
     @staticmethod
-    def forward(ctx, x, w1, w3):
+    def forward(ctx, x, w1, w3, clamp=None):
         K, N = x.shape[-1], w1.shape[0]
         x2 = x.reshape(-1, K)
         if x2.stride(1) != 1 or x2.stride(0) % 8 or x2.data_ptr() % 16:
@@ -1105,11 +1106,11 @@ class _GateUpSwiGLU(torch.autograd.Function):
         L = lib()
         if not getattr(L, "_swiglu_gemm_declared", False):
             vp, i32, i64 = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong
-            L.ttb_gemm_swiglu_bf16_2sm.argtypes = [vp, vp, vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, vp, vp]
+            L.ttb_gemm_swiglu_bf16_2sm.argtypes = [vp, vp, vp, vp, vp, vp, i32, i32, i32, i64, i64, i64, ctypes.c_float, ctypes.c_float, vp, vp]
             L.ttb_gemm_swiglu_bf16_2sm.restype = i32
             L._swiglu_gemm_declared = True
         check(L.ttb_gemm_swiglu_bf16_2sm(x2.data_ptr(), w1.data_ptr(), w3.data_ptr(), h.data_ptr(), _ptr(g), _ptr(u), M, N, K, x2.stride(0), w1.stride(0), N,
-                                         err_word(x.device).data_ptr(), stream_ptr()), f"gate/up GEMM + SwiGLU M={M} N={N} K={K}")
+                                         *(clamp or (0.0, 0.0)), err_word(x.device).data_ptr(), stream_ptr()), f"gate/up GEMM + SwiGLU M={M} N={N} K={K}")
         ctx.save_for_backward(x2, w1, w3, g, u)
         ctx.x_shape = x.shape
         return h.view(*x.shape[:-1], N)
@@ -1133,11 +1134,11 @@ class _GateUpSwiGLU(torch.autograd.Function):
             dx = gemm(dg, w1, b_mn=True)
             gemm(du, w3, b_mn=True, out=dx, accumulate=True)
             dx = dx.view(ctx.x_shape)
-        return dx, dw1, dw3
+        return dx, dw1, dw3, None
 
 
-def gate_up_swiglu(x: torch.Tensor, w1: torch.Tensor, w3: torch.Tensor) -> Optional[torch.Tensor]:
-    """Fused gate / up projections + SwiGLU, or ``None`` when the shapes do not suit the CTA-pair kernel (the caller then runs the three
+def gate_up_swiglu(x: torch.Tensor, w1: torch.Tensor, w3: torch.Tensor, clamp: Optional[Tuple[float, float]] = None) -> Optional[torch.Tensor]:
+    """Fused gate / up projections + SwiGLU (``clamp`` ``(limit, alpha)``: the clamped gate, outside autograd), or ``None`` when the shapes do not suit the CTA-pair kernel (the caller then runs the three
     separate operators)."""
     if not _PAIR_KERNEL or os.environ.get("TTB_FUSE_SWIGLU", "1") == "0":
         return None
@@ -1147,12 +1148,14 @@ def gate_up_swiglu(x: torch.Tensor, w1: torch.Tensor, w3: torch.Tensor) -> Optio
         return None
     if w1.data_ptr() % 16 or w3.data_ptr() % 16:
         return None
+    if clamp is not None and (clamp[0] <= 0.0 or (torch.is_grad_enabled() and (x.requires_grad or w1.requires_grad or w3.requires_grad))):
+        return None
     global _SM_PAIRS
     if _SM_PAIRS is None:
         _SM_PAIRS = max(1, torch.cuda.get_device_properties(x.device).multi_processor_count // 2)
     if K < 128 or (-(-M // 256)) * (-(-N // 128)) < _SM_PAIRS:
         return None
-    return _GateUpSwiGLU.apply(x, w1, w3)
+    return _GateUpSwiGLU.apply(x, w1, w3, clamp)
 
 
 def swiglu(gate: torch.Tensor, up: torch.Tensor) -> torch.Tensor:

@@ -111,9 +111,23 @@ def _declare(L: ctypes.CDLL) -> None:
     L.ttb_latent_value.argtypes = [vp, vp, vp, vp, i64, vp, i32, i32, i32, i32, i32, vp]
     L.ttb_latent_combine.argtypes = [vp, vp, vp, i32, i32, i32, i32, i32, vp]
     L.ttb_latent_gate_rows.argtypes = [vp, vp, i64, vp, i32, i32, i32, vp]
-    L.ttb_latent_attention_any.argtypes = [vp, i64, i64, i64, vp, i64, i64, i64, vp, i64, i64, vp, i64, i64, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32,
+    L.ttb_latent_attention_any.argtypes = [vp, i64, i64, i64, vp, i64, i64, i64, vp, i64, i64, vp, i64, i64, i64, vp, vp, vp, i64, i32, i32, i32, i32, i32, i32, i32, i32, i32, i32,
                                            vp, i32, vp, i64, i64, vp, i64, i64, f32, i32, vp]
     L.ttb_latent_decode_tile.argtypes = [i32, i32, i32]
+    L.ttb_span_decode_tile.argtypes = [i32, i32, i32]
+    L.ttb_span_prepare.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, f32, f32, i32, i32, vp]
+    L.ttb_span_prefill.argtypes = [vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, i32, i32, vp, i64, i64, vp, i64, i64, f32, vp, vp]
+    L.ttb_span_decode.argtypes = [vp, i64, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, i32, vp, i64, vp, i64, f32, vp, vp]
+    L.ttb_stream_step.argtypes = [vp, i32, vp, vp, vp, vp, vp, vp, vp, vp, i32, i32, i32, f32, f32, i32, i32, vp]
+    L.ttb_embed_positions.argtypes = [vp, vp, vp, vp, vp, i64, i32, i64, i64, i32, vp]
+    L.ttb_clamped_glu.argtypes = [vp, vp, vp, i64, i32, i64, i64, f32, f32, i32, vp]
+    L.ttb_lightning_recurrent.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, i32, i32, i32, i32, i32, i32, vp, i32, i32, vp]
+    L.ttb_lightning_chunks.argtypes = [vp, i64, vp, i64, vp, i64, vp, vp, vp, vp, vp, i32, i32, i32, i32, i32, i32, i32, vp, i32, vp, vp]
+    L.ttb_silu_rows.argtypes = [vp, i64, i64, i32, vp]
+    L.ttb_gated_norm.argtypes = [vp, i32, vp, vp, i64, vp, i64, i32, f32, i32, vp]
+    for fn in (L.ttb_span_decode_tile, L.ttb_span_prepare, L.ttb_span_prefill, L.ttb_span_decode, L.ttb_stream_step, L.ttb_embed_positions, L.ttb_clamped_glu, L.ttb_lightning_recurrent,
+               L.ttb_lightning_chunks, L.ttb_silu_rows, L.ttb_gated_norm):
+        fn.restype = i32
     for fn in (L.ttb_residual_norm, L.ttb_softcap, L.ttb_latent_decode_tile, L.ttb_latent_prefill, L.ttb_latent_decode, L.ttb_latent_prepare, L.ttb_latent_absorb, L.ttb_latent_value, L.ttb_latent_combine,
                L.ttb_latent_gate_rows, L.ttb_latent_attention_any):
         fn.restype = i32

@@ -89,6 +89,23 @@ inline int make_tmap_3d(CUtensorMap* out, const void* base, CUtensorMapDataType 
   return r == CUDA_SUCCESS ? kOk : kErrDriver;
 }
 
+// 4-D tensor [d3, d2, d1, d0] (d0 innermost, contiguous) with byte strides for the outer dimensions.
+inline int make_tmap_4d(CUtensorMap* out, const void* base, CUtensorMapDataType dt, const uint64_t (&d)[4], const uint64_t (&stride_bytes)[3],
+                        const uint32_t (&box_dims)[4], CUtensorMapSwizzle swz) {
+  EncodeTiledFn fn = encode_tiled_fn();
+  if (!fn) return kErrDriver;
+  if (reinterpret_cast<uintptr_t>(base) & 15) return kErrBadShape;
+  for (uint64_t s : stride_bytes)
+    if (s & 15) return kErrBadShape;
+  cuuint64_t dims[4] = {d[0], d[1], d[2], d[3]};
+  cuuint64_t strides[3] = {stride_bytes[0], stride_bytes[1], stride_bytes[2]};
+  cuuint32_t box[4] = {box_dims[0], box_dims[1], box_dims[2], box_dims[3]};
+  cuuint32_t estr[4] = {1, 1, 1, 1};
+  CUresult r = fn(out, dt, 4, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE, swz,
+                  CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+  return r == CUDA_SUCCESS ? kOk : kErrDriver;
+}
+
 inline int sm_count() {
   static int n = 0;
   if (!n) {

@@ -525,8 +525,11 @@ extern "C" int ttb_rmsnorm_bwd_noalloc(const void* dy, const void* x, const void
 extern "C" unsigned int ttb_violations_embedding(int reset);
 extern "C" unsigned int ttb_violations_loss(int reset);
 extern "C" unsigned int ttb_violations_latent(int reset);
+extern "C" unsigned int ttb_violations_streams(int reset);
+extern "C" unsigned int ttb_violations_span(int reset);
 
 // Out-of-range user indices (token ids, labels, positions) that kernels replaced by a safe value since the last reset.
 extern "C" unsigned int ttb_index_violations(int reset) {
-  return ttb_violations_rope(reset) + ttb_violations_embedding(reset) + ttb_violations_loss(reset) + ttb_violations_latent(reset);
+  return ttb_violations_rope(reset) + ttb_violations_embedding(reset) + ttb_violations_loss(reset) + ttb_violations_latent(reset) +
+         ttb_violations_streams(reset) + ttb_violations_span(reset);
 }

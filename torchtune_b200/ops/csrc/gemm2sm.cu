@@ -54,6 +54,7 @@ struct Params {
   int tma_store;
   int group_m;  // pair-tiles in m per scheduling group
   int tile_mult;  // 1, or an odd multiplier coprime to the tile count: tile t is replaced by (t · tile_mult) mod tiles (debug aid)
+  float glu_limit, glu_alpha;  // SWIGLU form, limit > 0: g·sigmoid(alpha·g)·(u + 1) with both pre-activations clamped, instead of silu(g)·u
   int save_gate_up;  // SWIGLU form: also store the two pre-activations (the backward pass needs them)
   int* err;
 };
@@ -320,7 +321,12 @@ gemm2sm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 // round the pre-activations to bf16 first: the unfused path computes SwiGLU from the stored bf16 values
                 g[i] = __bfloat162float(__float2bfloat16_rn(__uint_as_float(rg[j * 8 + i])));
                 u[i] = __bfloat162float(__float2bfloat16_rn(__uint_as_float(ru[j * 8 + i])));
-                o[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
+                if (p.glu_limit > 0.f) {
+                  const float gc = fminf(g[i], p.glu_limit), uc = fminf(fmaxf(u[i], -p.glu_limit), p.glu_limit);
+                  o[i] = gc / (1.f + __expf(-p.glu_alpha * gc)) * (uc + 1.f);
+                } else {
+                  o[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
+                }
               }
               const int chunk = (h * 4 + j) ^ (lane & 7);
               uint4 v;
@@ -606,9 +612,10 @@ extern "C" int ttb_gemm_bf16_dual_2sm(const void* A, const void* B, const void* 
 
 // Gated MLP up-projection with the activation in the epilogue: H[M, N] = silu(X · W1ᵀ) ⊙ (X · W3ᵀ) with X [M, K], W1 and W3 [N, K]
 // (row pitches lda, ldb; all bf16).  gate_out / up_out (both or neither; [M, N], row pitch ldc) receive the two pre-activations
-// rounded to bf16, which is what the backward pass of the unfused form would have read.
+// rounded to bf16, which is what the backward pass of the unfused form would have read.  glu_limit > 0: the gate is
+// g·sigmoid(glu_alpha·g)·(u + 1) with g clamped from above and u from both sides, instead of silu(g)·u.
 extern "C" int ttb_gemm_swiglu_bf16_2sm(const void* X, const void* W1, const void* W3, void* H, void* gate_out, void* up_out, int M, int N, int K,
-                                        long long lda, long long ldb, long long ldc, int* err, void* stream) {
+                                        long long lda, long long ldb, long long ldc, float glu_limit, float glu_alpha, int* err, void* stream) {
   using namespace ttb;
   if (M <= 0 || N <= 0 || K <= 0) return kErrBadShape;
   if ((lda & 7) || (ldb & 7) || (ldc & 7) || (N & 7) || (K & 7)) return kErrBadShape;
@@ -617,6 +624,7 @@ extern "C" int ttb_gemm_swiglu_bf16_2sm(const void* X, const void* W1, const voi
   p.M = M, p.N = N, p.K = K, p.C = H, p.ldc = ldc, p.bias = nullptr, p.alpha = 1.f;
   p.residual = nullptr, p.ldr = 0;
   p.accumulate = 0, p.tma_store = 1, p.save_gate_up = 0, p.tile_mult = 1, p.err = err, p.K2 = 0;
+  p.glu_limit = glu_limit, p.glu_alpha = glu_alpha;
   p.group_m = g2::group_setting();
   return g2::launch<false, false, true>(X, W1, W3, gate_out, up_out, p, lda, ldb, static_cast<cudaStream_t>(stream));
 }

@@ -16,6 +16,10 @@
 //   columns, N = heads).  Heads sit in the N dimension, so 16 heads cost 16 columns rather than a padded 128-row tile.  Cache
 //   rows are cut over CTAs (split keys); the partial outputs are combined by the value projection.
 //
+// Grouped-query attention over a key/value cache is the same pair of kernels without the two-part key: in prefill the second key part is
+// empty and `group` query heads read one key head; in decode the scores come from the keys alone (the second operand of the latent form,
+// up to 256 columns) and the pieces are the values.
+//
 // Row bounds: key j is visible to query i of batch row b iff lo(b, i) <= j <= hi(b, i), by default 0 <= j <= slot(i).  Every wait is
 // bounded and reports through the error word.
 #include "common/attn_math.cuh"
@@ -32,6 +36,7 @@ __device__ __forceinline__ float sigmoid_of(float z) { return 1.f / (1.f + __exp
 // ===================================================================================== prefill
 struct PrefillParams {
   int b, s, sk, heads;
+  int group;          // query heads per head of tmKn / tmV
   int slot0;          // cache slot of query 0 (sk = slot0 + s keys exist)
   int dim_panels, rot_panels, v_panels;
   int dim_steps, rot_steps;  // contraction steps of 16 columns
@@ -76,7 +81,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
   const int h = blockIdx.y, bi = blockIdx.z;
   const int q0 = (gridDim.x - 1 - blockIdx.x) * 2 * kBlk;  // the longest rows of a causal pattern start first
   const int row_base = bi * p.s;
-  const int krow_base = bi * p.sk;
+  const int hk = h / p.group;
   auto lo_of = [&](int i) { return p.lo != nullptr ? p.lo[bi * p.lo_row + i * p.lo_query] : 0; };
   auto hi_of = [&](int i) { return p.hi != nullptr ? p.hi[bi * p.hi_row + i * p.hi_query] : p.slot0 + i; };
 
@@ -148,8 +153,8 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       if (lane == 0) {
         uint8_t* dst = sK + ks * q_bytes;
         mbar_arrive_expect_tx(&k_full[ks], q_bytes);
-        for (int j = 0; j < p.dim_panels; ++j) tma_load_3d(dst + j * kPanelBytes, &tmKn, &k_full[ks], j * 64, h, krow_base + kv0);
-        for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(dst + (p.dim_panels + j) * kPanelBytes, &tmKr, &k_full[ks], j * 64, kv0, bi);
+        for (int j = 0; j < p.dim_panels; ++j) tma_load_4d(dst + j * kPanelBytes, &tmKn, &k_full[ks], j * 64, hk, kv0, bi);
+        for (int j = 0; j < p.rot_panels; ++j) tma_load_4d(dst + (p.dim_panels + j) * kPanelBytes, &tmKr, &k_full[ks], j * 64, 0, kv0, bi);
       }
       __syncwarp();
       if (!mbar_wait(&v_empty[vs], vph ^ 1)) {
@@ -159,7 +164,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
       if (lane == 0) {
         uint8_t* dst = sV + vs * v_bytes;
         mbar_arrive_expect_tx(&v_full[vs], v_bytes);
-        for (int j = 0; j < p.v_panels; ++j) tma_load_3d(dst + j * kPanelBytes, &tmV, &v_full[vs], j * 64, h, krow_base + kv0);
+        for (int j = 0; j < p.v_panels; ++j) tma_load_4d(dst + j * kPanelBytes, &tmV, &v_full[vs], j * 64, hk, kv0, bi);
       }
       __syncwarp();
       if (++ks == p.k_stages) ks = 0, kph ^= 1;
@@ -390,7 +395,9 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap tmQn, const __grid_con
 // ===================================================================================== decode
 struct DecodeParams {
   int b, heads, rank, rot, slots;
-  int pairs;       // 128-column pieces of the latent
+  int group, group_ctas;  // query heads that share keys, CTAs they take
+  int pairs;       // 128-column pieces of the latent (grouped form: of the values)
+  int q_panels;    // query panels multiplied with the pieces (grouped form: none)
   int c_steps, rot_panels, rot_steps;
   int ring;        // 32 KB slots for pieces
   int rot_stages;
@@ -463,7 +470,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   uint8_t* sC = smem;                                        // [ring] pieces: KB rows x 128 columns
   uint8_t* sR = sC + p.ring * kPairBytes;                    // [rot_stages]
   uint8_t* sQ = sR + p.rot_stages * p.rot_panels * kKeyPanel;  // 2 * pairs latent panels, then the rotated ones
-  uint8_t* sP = sQ + (2 * p.pairs + p.rot_panels) * kQPanel;     // [2] tiles of [HN heads, KB keys]
+  uint8_t* sP = sQ + (p.q_panels + p.rot_panels) * kQPanel;     // [2] tiles of [HN heads, KB keys]
   uint64_t* bars = reinterpret_cast<uint64_t*>(sP + 2 * kPBytes);
   uint64_t* c_full = bars;                 // [ring]
   uint64_t* c_empty = bars + kMaxRing;     // [ring]
@@ -479,7 +486,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   float* s_red = reinterpret_cast<float*>(tmem_slot + 2);  // [4][HN]
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int split = blockIdx.x, splits = gridDim.x, h0 = blockIdx.y * HN, bi = blockIdx.z;
+  const int split = blockIdx.x, splits = gridDim.x, bi = blockIdx.z;
+  const int hk = blockIdx.y / p.group_ctas, h0 = hk * p.group + (blockIdx.y % p.group_ctas) * HN, h_end = (hk + 1) * p.group;
   const int newest = p.slot != nullptr ? *p.slot : p.slot_host;
   const int hi = min(p.hi != nullptr ? p.hi[bi * p.hi_row] : newest, p.slots - 1);
   const int lo = max(p.lo != nullptr ? p.lo[bi * p.lo_row] : 0, 0);
@@ -519,9 +527,9 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   if (warp == 0) {
     // ---------------------------------------------------------------- TMA producer
     if (lane == 0 && n_blocks > 0) {
-      mbar_arrive_expect_tx(q_full, (2 * p.pairs + p.rot_panels) * kQPanel);
-      for (int j = 0; j < 2 * p.pairs; ++j) tma_load_3d(sQ + j * kQPanel, &tmQ, q_full, j * 64, h0, bi);
-      for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(sQ + (2 * p.pairs + j) * kQPanel, &tmQ, q_full, p.rank + j * 64, h0, bi);
+      mbar_arrive_expect_tx(q_full, (p.q_panels + p.rot_panels) * kQPanel);
+      for (int j = 0; j < p.q_panels; ++j) tma_load_3d(sQ + j * kQPanel, &tmQ, q_full, j * 64, h0, bi);
+      for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(sQ + (p.q_panels + j) * kQPanel, &tmQ, q_full, (p.q_panels > 0 ? p.rank : 0) + j * 64, h0, bi);
     }
     int cs = 0, rs = 0;
     uint32_t cph = 0, rph = 0;
@@ -532,8 +540,8 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
         ok = mbar_wait(&c_empty[cs], cph ^ 1);
         if (ok && lane == 0) {
           mbar_arrive_expect_tx(&c_full[cs], kPairBytes);
-          tma_load_3d(sC + cs * kPairBytes, &tmC, &c_full[cs], u * 128, key0, bi);
-          tma_load_3d(sC + cs * kPairBytes + kKeyPanel, &tmC, &c_full[cs], u * 128 + 64, key0, bi);
+          tma_load_4d(sC + cs * kPairBytes, &tmC, &c_full[cs], u * 128, hk, key0, bi);
+          tma_load_4d(sC + cs * kPairBytes + kKeyPanel, &tmC, &c_full[cs], u * 128 + 64, hk, key0, bi);
         }
         __syncwarp();
         if (++cs == p.ring) cs = 0, cph ^= 1;
@@ -546,7 +554,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       if (lane == 0) {
         uint8_t* dst = sR + rs * p.rot_panels * kKeyPanel;
         mbar_arrive_expect_tx(&r_full[rs], p.rot_panels * kKeyPanel);
-        for (int j = 0; j < p.rot_panels; ++j) tma_load_3d(dst + j * kKeyPanel, &tmR, &r_full[rs], j * 64, key0, bi);
+        for (int j = 0; j < p.rot_panels; ++j) tma_load_4d(dst + j * kKeyPanel, &tmR, &r_full[rs], j * 64, hk, key0, bi);
       }
       __syncwarp();
       if (++rs == p.rot_stages) rs = 0, rph ^= 1;
@@ -563,7 +571,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       const int st = it & 1;
       const uint32_t tS = tmem_base + st * HN;
       ok = mbar_wait(&s_free[st], ((it >> 1) & 1) ^ 1);
-      for (int u = 0; u < p.pairs && ok; ++u) {
+      for (int u = 0; 2 * u < p.q_panels && ok; ++u) {
         ok = mbar_wait(&c_full[cs], cph);
         tc_fence_after();
         if (ok && elect_one()) {
@@ -579,7 +587,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tc_fence_after();
       if (ok && elect_one()) {
         for (int j = 0; j < p.rot_panels; ++j)
-          umma_panel(tS, dR + (rs * p.rot_panels + j) * (kKeyPanel >> 4), dQ + (2 * p.pairs + j) * (kQPanel >> 4), p.rot_steps - 4 * j, idesc, true);
+          umma_panel(tS, dR + (rs * p.rot_panels + j) * (kKeyPanel >> 4), dQ + (p.q_panels + j) * (kQPanel >> 4), p.rot_steps - 4 * j, idesc, p.q_panels > 0 || j > 0);
         umma_commit(&r_empty[rs]);
         umma_commit(&s_full[st]);
       }
@@ -712,7 +720,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     const long long row0 = (static_cast<long long>(split) * p.b + bi) * p.heads + h0;
 #pragma unroll
     for (int h = 0; h < HN; ++h)
-      if (r == h && h0 + h < p.heads) p.ml[row0 + h] = make_float2(m[h], s_red[h] + s_red[HN + h] + s_red[2 * HN + h] + s_red[3 * HN + h]);
+      if (r == h && h0 + h < h_end) p.ml[row0 + h] = make_float2(m[h], s_red[h] + s_red[HN + h] + s_red[2 * HN + h] + s_red[3 * HN + h]);
     if (n_blocks > 0 && ok) {
 #pragma unroll 1
       for (int u = 0; u < p.pairs; ++u) {
@@ -724,7 +732,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
           float* dst = p.o + row0 * p.rank + col;
 #pragma unroll
           for (int h = 0; h < HN; ++h)
-            if (h0 + h < p.heads) dst[static_cast<long long>(h) * p.rank] = __uint_as_float(v[h]);
+            if (h0 + h < h_end) dst[static_cast<long long>(h) * p.rank] = __uint_as_float(v[h]);
         }
       }
     }
@@ -738,6 +746,12 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
 
 static constexpr int kSmemLimit = 227 * 1024;
 
+// rows of 64-column panels: [batch, keys, heads, columns] with the given row, head and batch pitches
+static int map4(CUtensorMap* m, const void* base, uint64_t cols, uint64_t heads, uint64_t keys, uint64_t batch, uint64_t head_pitch, uint64_t key_pitch, uint64_t batch_pitch,
+                uint32_t box_keys) {
+  return make_tmap_4d(m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, {cols, heads, keys, batch}, {head_pitch * 2, key_pitch * 2, batch_pitch * 2}, {64, 1, box_keys, 1},
+                      CU_TENSOR_MAP_SWIZZLE_128B);
+}
 static int map3(CUtensorMap* m, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1_elems, uint64_t s2_elems, uint32_t b1, uint32_t b2) {
   return make_tmap_3d(m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, d0, d1, d2, s1_elems * 2, s2_elems * 2, 64, b1, b2, CU_TENSOR_MAP_SWIZZLE_128B);
 }
@@ -746,7 +760,7 @@ static int map3(CUtensorMap* m, const void* base, uint64_t d0, uint64_t d1, uint
 template <int HN, int KB>
 static int plan_decode(DecodeParams& p) {
   const int q_panel = HN * 128, key_panel = KB * 128;
-  const int fixed = (2 * p.pairs + p.rot_panels + 2 * (KB / 64)) * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
+  const int fixed = (p.q_panels + p.rot_panels + 2 * (KB / 64)) * q_panel + 1024 + (kDecodeBarriers + 2) * 8 + 4 * HN * 4;
   const int rot_bytes = p.rot_panels * key_panel;
   p.rot_stages = fixed + 2 * rot_bytes + 2 * p.pairs * 2 * key_panel <= kSmemLimit ? 2 : 1;
   int ring = (kSmemLimit - fixed - p.rot_stages * rot_bytes) / (2 * key_panel);
@@ -763,34 +777,72 @@ static bool small_tiles(DecodeParams p) {
   return !p.lookahead;
 }
 
+// What the decode kernel reads: queries [b, heads, q_width] with a batch pitch, pieces and second operand as [b, slots, key heads, columns].
+struct DecodeInputs {
+  const void* q;
+  uint64_t q_width, q_batch;
+  const void* c;
+  uint64_t c_head, c_key, c_batch;
+  const void* r;
+  uint64_t r_head, r_key, r_batch;
+  int key_heads;
+};
+
 template <int HN, int KB>
-static int launch_decode(DecodeParams& p, const void* q, const void* cache, int splits, cudaStream_t st) {
+static int launch_decode(DecodeParams& p, const DecodeInputs& in, int splits, cudaStream_t st) {
   const int smem = plan_decode<HN, KB>(p);
   if (p.ring < p.pairs || smem > kSmemLimit) return kErrTooLarge;
   int cols = 32;
   while (cols < 2 * HN + p.pairs * HN) cols *= 2;
   p.tmem_cols = cols;
-  const long long row = p.rank + p.rot;
+  p.group_ctas = (p.group + HN - 1) / HN;
   CUtensorMap tq, tc, tr;
   int rc;
-  if ((rc = map3(&tq, q, row, p.heads, p.b, row, row * p.heads, HN, 1)) != kOk) return rc;
-  if ((rc = map3(&tc, cache, p.rank, p.slots, p.b, row, row * p.slots, KB, 1)) != kOk) return rc;
-  if ((rc = map3(&tr, static_cast<const __nv_bfloat16*>(cache) + p.rank, p.rot, p.slots, p.b, row, row * p.slots, KB, 1)) != kOk) return rc;
+  if ((rc = map3(&tq, in.q, in.q_width, p.heads, p.b, in.q_width, in.q_batch, HN, 1)) != kOk) return rc;
+  if ((rc = map4(&tc, in.c, p.rank, in.key_heads, p.slots, p.b, in.c_head, in.c_key, in.c_batch, KB)) != kOk) return rc;
+  if ((rc = map4(&tr, in.r, p.rot, in.key_heads, p.slots, p.b, in.r_head, in.r_key, in.r_batch, KB)) != kOk) return rc;
   static bool attr = false;
   if (!attr) {
     if (cudaFuncSetAttribute(latent_decode_kernel<HN, KB>, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit) != cudaSuccess) return kErrDriver;
     attr = true;
   }
   TTB_COUNT_LAUNCH(1);
-  latent_decode_kernel<HN, KB><<<dim3(splits, (p.heads + HN - 1) / HN, p.b), kDecodeThreads, smem, st>>>(tq, tc, tr, p);
+  latent_decode_kernel<HN, KB><<<dim3(splits, in.key_heads * p.group_ctas, p.b), kDecodeThreads, smem, st>>>(tq, tc, tr, p);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 
-static DecodeParams decode_shape(int heads, int rank, int rot) {
+static int launch_decode_any(DecodeParams& p, const DecodeInputs& in, int splits, cudaStream_t st) {
+  if (p.group <= 16) return small_tiles<16>(p) ? launch_decode<16, 64>(p, in, splits, st) : launch_decode<16, 128>(p, in, splits, st);
+  return small_tiles<32>(p) ? launch_decode<32, 64>(p, in, splits, st) : launch_decode<32, 128>(p, in, splits, st);
+}
+
+// `pieces_score`: the pieces are keys as well as values (latents)
+static DecodeParams decode_shape(int heads, int group, int rank, int rot, bool pieces_score) {
   DecodeParams p{};
-  p.heads = heads, p.rank = rank, p.rot = rot;
-  p.pairs = (rank + 127) / 128, p.c_steps = (rank + 15) / 16, p.rot_panels = (rot + 63) / 64, p.rot_steps = (rot + 15) / 16;
+  p.heads = heads, p.group = group, p.rank = rank, p.rot = rot;
+  p.pairs = (rank + 127) / 128, p.q_panels = pieces_score ? 2 * p.pairs : 0, p.c_steps = (rank + 15) / 16, p.rot_panels = (rot + 63) / 64, p.rot_steps = (rot + 15) / 16;
   return p;
+}
+
+static int launch_prefill(PrefillParams& p, int dim, int rot, const CUtensorMap& tqn, const CUtensorMap& tqr, const CUtensorMap& tkn, const CUtensorMap& tkr, const CUtensorMap& tv,
+                          cudaStream_t st) {
+  p.dim_panels = (dim + 63) / 64, p.rot_panels = (rot + 63) / 64, p.v_panels = (p.vdim + 63) / 64;
+  p.dim_steps = (dim + 15) / 16, p.rot_steps = (rot + 15) / 16;
+  const int kp = p.dim_panels + p.rot_panels;
+  if (p.v_panels > 2 || kp > 4) return kErrTooLarge;
+  p.k_stages = p.v_stages = 2;
+  if (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels > 14) p.v_stages = 1;
+  if (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels > 14) p.k_stages = 1;
+  const int smem = (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels) * kPanelBytes + 1024 + 256;
+  if (smem > kSmemLimit) return kErrTooLarge;
+  static bool attr = false;
+  if (!attr) {
+    if (cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit) != cudaSuccess) return kErrDriver;
+    attr = true;
+  }
+  TTB_COUNT_LAUNCH(1);
+  latent_prefill_kernel<<<dim3((p.s + 2 * kBlk - 1) / (2 * kBlk), p.heads, p.b), kPrefillThreads, smem, st>>>(tqn, tqr, tkn, tkr, tv, p);
+  return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 
 }  // namespace latent
@@ -808,34 +860,39 @@ extern "C" int ttb_latent_prefill(const void* q, long long ld_q, const void* kn,
   if (b <= 0 || s <= 0 || heads <= 0 || sk < slot0 + s || slot0 < 0) return kErrBadShape;
   if ((dim & 7) || (rot & 7) || (vdim & 7) || dim <= 0 || rot <= 0 || vdim <= 0 || (gate != nullptr && ((gate_ld & 7) || (reinterpret_cast<uintptr_t>(gate) & 15)))) return kErrBadShape;
   PrefillParams p{};
-  p.b = b, p.s = s, p.sk = sk, p.heads = heads, p.slot0 = slot0, p.vdim = vdim, p.scale = scale;
-  p.dim_panels = (dim + 63) / 64, p.rot_panels = (rot + 63) / 64, p.v_panels = (vdim + 63) / 64;
-  p.dim_steps = (dim + 15) / 16, p.rot_steps = (rot + 15) / 16;
-  const int kp = p.dim_panels + p.rot_panels;
-  if (p.v_panels > 2 || kp > 4) return kErrTooLarge;
-  p.k_stages = p.v_stages = 2;
-  if (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels > 14) p.v_stages = 1;
-  if (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels > 14) p.k_stages = 1;
-  const int smem = (2 * kp + p.k_stages * kp + p.v_stages * p.v_panels) * kPanelBytes + 1024 + 256;
-  if (smem > kSmemLimit) return kErrTooLarge;
+  p.b = b, p.s = s, p.sk = sk, p.heads = heads, p.group = 1, p.slot0 = slot0, p.vdim = vdim, p.scale = scale;
   p.lo = lo, p.lo_row = lo_row, p.lo_query = lo_query, p.hi = hi, p.hi_row = hi_row, p.hi_query = hi_query;
   p.gate = static_cast<const __nv_bfloat16*>(gate), p.gate_ld = gate_ld, p.o = static_cast<__nv_bfloat16*>(o), p.err = err;
   CUtensorMap tqn, tqr, tkn, tkr, tv;
-  const uint64_t tq = static_cast<uint64_t>(b) * s, tk = static_cast<uint64_t>(b) * sk;
+  const uint64_t tq = static_cast<uint64_t>(b) * s;
   int rc;
   if ((rc = map3(&tqn, q, dim, heads, tq, dim + rot, ld_q, 1, kBlk)) != kOk) return rc;
   if ((rc = map3(&tqr, static_cast<const __nv_bfloat16*>(q) + dim, rot, heads, tq, dim + rot, ld_q, 1, kBlk)) != kOk) return rc;
-  if ((rc = map3(&tkn, kn, dim, heads, tk, dim, ld_kn, 1, kBlk)) != kOk) return rc;
-  if ((rc = map3(&tkr, kr, rot, sk, b, ld_kr, kr_batch, kBlk, 1)) != kOk) return rc;
-  if ((rc = map3(&tv, v, vdim, heads, tk, vdim, ld_v, 1, kBlk)) != kOk) return rc;
-  static bool attr = false;
-  if (!attr) {
-    if (cudaFuncSetAttribute(latent_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, kSmemLimit) != cudaSuccess) return kErrDriver;
-    attr = true;
-  }
-  TTB_COUNT_LAUNCH(1);
-  latent_prefill_kernel<<<dim3((s + 2 * kBlk - 1) / (2 * kBlk), heads, b), kPrefillThreads, smem, static_cast<cudaStream_t>(stream)>>>(tqn, tqr, tkn, tkr, tv, p);
-  return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
+  if ((rc = map4(&tkn, kn, dim, heads, sk, b, dim, ld_kn, sk * ld_kn, kBlk)) != kOk) return rc;
+  if ((rc = map4(&tkr, kr, rot, 1, sk, b, ld_kr, ld_kr, kr_batch, kBlk)) != kOk) return rc;
+  if ((rc = map4(&tv, v, vdim, heads, sk, b, vdim, ld_v, sk * ld_v, kBlk)) != kOk) return rc;
+  return launch_prefill(p, dim, rot, tqn, tqr, tkn, tkr, tv, static_cast<cudaStream_t>(stream));
+}
+
+// Grouped-query attention of many queries per sequence: q [b*s, ld_q] with head h at column h*dim; k [b, slots, key_heads, dim] and
+// v [b, slots, key_heads, vdim], of which the first sk slots exist; o [b*s, heads*vdim].  heads is a multiple of key_heads.
+extern "C" int ttb_span_prefill(const void* q, long long ld_q, const void* k, const void* v, void* o, int b, int s, int sk, int slots, int heads, int key_heads, int dim, int vdim,
+                                int slot0, const int* lo, long long lo_row, long long lo_query, const int* hi, long long hi_row, long long hi_query, float scale, int* err, void* stream) {
+  using namespace ttb;
+  using namespace ttb::latent;
+  if (b <= 0 || s <= 0 || heads <= 0 || key_heads <= 0 || heads % key_heads || sk < slot0 + s || sk > slots || slot0 < 0) return kErrBadShape;
+  if ((dim & 7) || (vdim & 7) || dim <= 0 || vdim <= 0) return kErrBadShape;
+  PrefillParams p{};
+  p.b = b, p.s = s, p.sk = sk, p.heads = heads, p.group = heads / key_heads, p.slot0 = slot0, p.vdim = vdim, p.scale = scale;
+  p.lo = lo, p.lo_row = lo_row, p.lo_query = lo_query, p.hi = hi, p.hi_row = hi_row, p.hi_query = hi_query;
+  p.o = static_cast<__nv_bfloat16*>(o), p.err = err;
+  CUtensorMap tq, tk, tv;
+  const uint64_t k_row = static_cast<uint64_t>(key_heads) * dim, v_row = static_cast<uint64_t>(key_heads) * vdim;
+  int rc;
+  if ((rc = map3(&tq, q, dim, heads, static_cast<uint64_t>(b) * s, dim, ld_q, 1, kBlk)) != kOk) return rc;
+  if ((rc = map4(&tk, k, dim, key_heads, sk, b, dim, k_row, k_row * slots, kBlk)) != kOk) return rc;
+  if ((rc = map4(&tv, v, vdim, key_heads, sk, b, vdim, v_row, v_row * slots, kBlk)) != kOk) return rc;
+  return launch_prefill(p, dim, 0, tq, tq, tk, tk, tv, static_cast<cudaStream_t>(stream));
 }
 
 // One query per batch row, absorbed: q [b, heads, rank + rot], cache [b, slots, rank + rot] (bf16); o [splits, b, heads, rank] and
@@ -847,19 +904,44 @@ extern "C" int ttb_latent_decode(const void* q, const void* cache, float* o, flo
   using namespace ttb::latent;
   if (b <= 0 || heads <= 0 || slots <= 0 || splits <= 0 || (rank & 7) || (rot & 7) || rank <= 0 || rot <= 0) return kErrBadShape;
   if (rank > 512 || rot > 128) return kErrTooLarge;
-  DecodeParams p = decode_shape(heads, rank, rot);
+  DecodeParams p = decode_shape(heads, heads, rank, rot, true);
   p.b = b, p.slots = slots, p.scale = scale;
   p.slot = slot, p.slot_host = slot_host, p.lo = lo, p.lo_row = lo_row, p.hi = hi, p.hi_row = hi_row;
   p.o = o, p.ml = reinterpret_cast<float2*>(ml), p.err = err;
-  auto st = static_cast<cudaStream_t>(stream);
-  if (heads <= 16) return small_tiles<16>(p) ? launch_decode<16, 64>(p, q, cache, splits, st) : launch_decode<16, 128>(p, q, cache, splits, st);
-  return small_tiles<32>(p) ? launch_decode<32, 64>(p, q, cache, splits, st) : launch_decode<32, 128>(p, q, cache, splits, st);
+  const uint64_t row = rank + rot;
+  const DecodeInputs in{q, row, row * heads, cache, row, row, row * slots, static_cast<const __nv_bfloat16*>(cache) + rank, row, row, row * slots, 1};
+  return launch_decode_any(p, in, splits, static_cast<cudaStream_t>(stream));
+}
+
+// Grouped-query attention of one query per batch row: q [b, heads, dim] with row pitch ld_q, k [b, slots, key_heads, dim], v [b, slots, key_heads, vdim]
+// (bf16); o [splits, b, heads, vdim] and ml [splits, b, heads, 2] fp32 partial results.
+extern "C" int ttb_span_decode(const void* q, long long ld_q, const void* k, const void* v, float* o, float* ml, int b, int heads, int key_heads, int dim, int vdim, int slots, int splits,
+                               const int* slot, int slot_host, const int* lo, long long lo_row, const int* hi, long long hi_row, float scale, int* err, void* stream) {
+  using namespace ttb;
+  using namespace ttb::latent;
+  if (b <= 0 || heads <= 0 || key_heads <= 0 || heads % key_heads || slots <= 0 || splits <= 0 || (dim & 7) || (vdim & 7) || dim <= 0 || vdim <= 0) return kErrBadShape;
+  if (vdim > 512 || dim > 256) return kErrTooLarge;
+  DecodeParams p = decode_shape(heads, heads / key_heads, vdim, dim, false);
+  p.b = b, p.slots = slots, p.scale = scale;
+  p.slot = slot, p.slot_host = slot_host, p.lo = lo, p.lo_row = lo_row, p.hi = hi, p.hi_row = hi_row;
+  p.o = o, p.ml = reinterpret_cast<float2*>(ml), p.err = err;
+  const uint64_t k_row = static_cast<uint64_t>(key_heads) * dim, v_row = static_cast<uint64_t>(key_heads) * vdim;
+  const DecodeInputs in{q, static_cast<uint64_t>(dim), static_cast<uint64_t>(ld_q), v, static_cast<uint64_t>(vdim), v_row, v_row * slots, k, static_cast<uint64_t>(dim), k_row, k_row * slots, key_heads};
+  return launch_decode_any(p, in, splits, static_cast<cudaStream_t>(stream));
 }
 
 // Keys per tile of ttb_latent_decode for these sizes (a key range should not be shorter).
 extern "C" int ttb_latent_decode_tile(int heads, int rank, int rot) {
   using namespace ttb::latent;
   if (rank <= 0 || rank > 512 || rot <= 0 || rot > 128) return 128;
-  const DecodeParams p = decode_shape(heads, rank, rot);
+  const DecodeParams p = decode_shape(heads, heads, rank, rot, true);
   return (heads <= 16 ? small_tiles<16>(p) : small_tiles<32>(p)) ? 64 : 128;
+}
+
+// The same for ttb_span_decode, with the number of query heads that share a key head.
+extern "C" int ttb_span_decode_tile(int group, int dim, int vdim) {
+  using namespace ttb::latent;
+  if (group <= 0 || dim <= 0 || dim > 256 || vdim <= 0 || vdim > 512) return 128;
+  const DecodeParams p = decode_shape(group, group, vdim, dim, false);
+  return (group <= 16 ? small_tiles<16>(p) : small_tiles<32>(p)) ? 64 : 128;
 }

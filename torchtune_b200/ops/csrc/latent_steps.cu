@@ -290,7 +290,8 @@ __global__ void __launch_bounds__(256) latent_absorb_kernel(const T* __restrict_
 
 // ------------------------------------------------------------------------------- split-key partials
 // o [splits, R, heads, K] fp32 with ml [splits, R, heads] (log2-domain maximum, sum) -> the normalised rows, [R, heads, K] fp32 or
-// head-major [heads, R, K] bf16 (the row order of a grouped GEMM whose groups are heads).  One CTA per (row, head, 128 columns).
+// head-major [heads, R, K] bf16 (the row order of a grouped GEMM whose groups are heads), or [R, heads, K] bf16.  One CTA per (row, head,
+// 128 columns).
 __device__ __forceinline__ float warp_max_of(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, o));
@@ -298,7 +299,9 @@ __device__ __forceinline__ float warp_max_of(float v) {
 }
 
 // GROUPS groups of 128 threads, each adding up every GROUPS-th range: several when there are many ranges (few rows).
-template <bool HEAD_MAJOR, int GROUPS>
+enum CombineForm { kRowsF32 = 0, kHeadsBf16 = 1, kRowsBf16 = 2 };
+
+template <int FORM, int GROUPS>
 __global__ void __launch_bounds__(128 * GROUPS) latent_combine_kernel(const float* __restrict__ o, const float2* __restrict__ ml, void* __restrict__ out, int splits,
                                                                               int R, int heads, int K) {
   extern __shared__ float wts[];  // [splits]: exp2(m_s - m) / sum, 0 for a split without keys (which has written nothing)
@@ -342,7 +345,8 @@ __global__ void __launch_bounds__(128 * GROUPS) latent_combine_kernel(const floa
   if (group == 0 && k < K) {
 #pragma unroll
     for (int g = 1; g < GROUPS; ++g) acc += part[g][col];
-    if constexpr (HEAD_MAJOR) static_cast<__nv_bfloat16*>(out)[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(acc);
+    if constexpr (FORM == kRowsBf16) static_cast<__nv_bfloat16*>(out)[rh * K + k] = __float2bfloat16_rn(acc);
+    else if constexpr (FORM == kHeadsBf16) static_cast<__nv_bfloat16*>(out)[(static_cast<long long>(h) * R + r) * K + k] = __float2bfloat16_rn(acc);
     else static_cast<float*>(out)[rh * K + k] = acc;
   }
 }
@@ -448,6 +452,7 @@ struct AnyParams {
   const void* gate;
   long long gate_ld;
   int b, s, sk, heads, d1, d2, dv;
+  int group;       // query heads per key head (k1_h, v_h: pitch of key heads)
   int heads_as_rows, out_f32, key_tile;
   const int* slot;
   int slot_host;
@@ -460,7 +465,7 @@ struct AnyParams {
 
 static constexpr int kAnyRows = 16;
 
-// 128 threads, 16 rows per CTA: 16 queries of one head, or (heads_as_rows) 16 heads of one query when all heads share keys and values.
+// 128 threads, 16 rows per CTA: 16 queries of one head, or (heads_as_rows, one query per sequence) 16 of the heads that share a key head.
 template <typename T>
 __global__ void __launch_bounds__(128) latent_attention_any_kernel(AnyParams p) {
   extern __shared__ float sm[];
@@ -476,10 +481,10 @@ __global__ void __launch_bounds__(128) latent_attention_any_kernel(AnyParams p) 
   __shared__ int s_lo[kAnyRows], s_hi[kAnyRows];
   const int bi = blockIdx.z;
   const int row0 = blockIdx.x * kAnyRows;
-  const int n_rows = min(kAnyRows, (p.heads_as_rows ? p.heads : p.s) - row0);
-  auto query_of = [&](int r) { return p.heads_as_rows ? static_cast<int>(blockIdx.y) : row0 + r; };
-  auto head_of = [&](int r) { return p.heads_as_rows ? row0 + r : static_cast<int>(blockIdx.y); };
-  const int h_shared = p.heads_as_rows ? 0 : static_cast<int>(blockIdx.y);
+  const int n_rows = min(kAnyRows, (p.heads_as_rows ? p.group : p.s) - row0);
+  const int h_shared = p.heads_as_rows ? static_cast<int>(blockIdx.y) : static_cast<int>(blockIdx.y) / p.group;
+  auto query_of = [&](int r) { return p.heads_as_rows ? 0 : row0 + r; };
+  auto head_of = [&](int r) { return p.heads_as_rows ? h_shared * p.group + row0 + r : static_cast<int>(blockIdx.y); };
   const int slot0 = p.slot != nullptr ? *p.slot : p.slot_host;
 
   for (int t = threadIdx.x; t < kAnyRows * d; t += 128) {
@@ -665,20 +670,22 @@ extern "C" int ttb_latent_value(const float* o, const float* ml, const void* w, 
               : launch_value<__nv_bfloat16>(o, ml, w, gate, gate_ld, out, rows, heads, K, N, st);
 }
 
-// [rows, heads, K] fp32, or (head_major) [heads, rows, K] bf16
-extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, int splits, int rows, int heads, int K, int head_major, void* stream) {
-  if (rows <= 0 || heads <= 0 || K <= 0 || splits <= 0 || splits > 8192) return kErrBadShape;
+// form 0: [rows, heads, K] fp32, 1: [heads, rows, K] bf16, 2: [rows, heads, K] bf16
+extern "C" int ttb_latent_combine(const float* o, const float* ml, void* out, int splits, int rows, int heads, int K, int form, void* stream) {
+  if (rows <= 0 || heads <= 0 || K <= 0 || splits <= 0 || splits > 8192 || form < 0 || form > 2) return kErrBadShape;
   auto st = static_cast<cudaStream_t>(stream);
   auto m = reinterpret_cast<const float2*>(ml);
   TTB_COUNT_LAUNCH(1);
   const dim3 grid(rows, heads, (K + 127) / 128);
-#define TTB_COMBINE(HEAD_MAJOR, GROUPS) latent_combine_kernel<HEAD_MAJOR, GROUPS><<<grid, 128 * GROUPS, splits * 4, st>>>(o, m, out, splits, rows, heads, K)
+#define TTB_COMBINE(FORM, GROUPS) latent_combine_kernel<FORM, GROUPS><<<grid, 128 * GROUPS, splits * 4, st>>>(o, m, out, splits, rows, heads, K)
   if (splits < 8) {
-    if (head_major) TTB_COMBINE(true, 1);
-    else TTB_COMBINE(false, 1);
+    if (form == kRowsBf16) TTB_COMBINE(kRowsBf16, 1);
+    else if (form == kHeadsBf16) TTB_COMBINE(kHeadsBf16, 1);
+    else TTB_COMBINE(kRowsF32, 1);
   } else {
-    if (head_major) TTB_COMBINE(true, 4);
-    else TTB_COMBINE(false, 4);
+    if (form == kRowsBf16) TTB_COMBINE(kRowsBf16, 4);
+    else if (form == kHeadsBf16) TTB_COMBINE(kHeadsBf16, 4);
+    else TTB_COMBINE(kRowsF32, 4);
   }
 #undef TTB_COMBINE
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
@@ -698,12 +705,12 @@ extern "C" int ttb_latent_gate_rows(const void* x, const void* gate, long long g
 
 extern "C" int ttb_latent_attention_any(const void* q, long long q_b, long long q_i, long long q_h, const void* k1, long long k1_b, long long k1_j, long long k1_h,
                                         const void* k2, long long k2_b, long long k2_j, const void* v, long long v_b, long long v_j, long long v_h, void* o,
-                                        float* ml, const void* gate, long long gate_ld, int b, int s, int sk, int heads, int d1, int d2, int dv, int heads_as_rows,
-                                        int out_f32, const int* slot, int slot_host, const int* lo, long long lo_row, long long lo_query, const int* hi,
+                                        float* ml, const void* gate, long long gate_ld, int b, int s, int sk, int heads, int group, int d1, int d2, int dv,
+                                        int heads_as_rows, int out_f32, const int* slot, int slot_host, const int* lo, long long lo_row, long long lo_query, const int* hi,
                                         long long hi_row, long long hi_query, float scale, int wide, void* stream) {
-  if (b <= 0 || s <= 0 || sk <= 0 || heads <= 0 || d1 < 0 || d2 < 0 || d1 + d2 <= 0 || dv <= 0) return kErrBadShape;
+  if (b <= 0 || s <= 0 || sk <= 0 || heads <= 0 || group <= 0 || heads % group || d1 < 0 || d2 < 0 || d1 + d2 <= 0 || dv <= 0 || (heads_as_rows && s != 1)) return kErrBadShape;
   AnyParams p{q, q_b, q_i, q_h, k1, k1_b, k1_j, k1_h, k2, k2_b, k2_j, v, v_b, v_j, v_h, o, reinterpret_cast<float2*>(ml), gate, gate_ld,
-              b, s, sk, heads, d1, d2, dv, heads_as_rows, out_f32, 32, slot, slot_host, lo, lo_row, lo_query, hi, hi_row, hi_query, scale};
+              b, s, sk, heads, d1, d2, dv, group, heads_as_rows, out_f32, 32, slot, slot_host, lo, lo_row, lo_query, hi, hi_row, hi_query, scale};
   const int d = d1 + d2;
   auto need = [&](int kt) { return (kAnyRows * d + kt * (d + 1) + kt * dv + kAnyRows * dv + kAnyRows * kt + 3 * kAnyRows) * 4; };
   while (p.key_tile > 1 && need(p.key_tile) > kSmemMax - 1024) p.key_tile /= 2;
@@ -711,7 +718,7 @@ extern "C" int ttb_latent_attention_any(const void* q, long long q_b, long long 
   if (smem > kSmemMax - 1024) return kErrTooLarge;
   static int gf = 0, gb = 0;
   if (!(wide ? allow_smem(latent_attention_any_kernel<float>, smem, gf) : allow_smem(latent_attention_any_kernel<__nv_bfloat16>, smem, gb))) return kErrDriver;
-  const int rows = heads_as_rows ? heads : s, other = heads_as_rows ? s : heads;
+  const int rows = heads_as_rows ? group : s, other = heads_as_rows ? heads / group : heads;
   if (other > 65535 || b > 65535) return kErrTooLarge;
   const dim3 grid((rows + kAnyRows - 1) / kAnyRows, other, b);
   auto st = static_cast<cudaStream_t>(stream);

@@ -84,7 +84,7 @@ def prefill(q: torch.Tensor, kn: torch.Tensor, v: torch.Tensor, buf: torch.Tenso
                                        _p(bounds.hi), bounds.hi_row, bounds.hi_query, float(scale), err_word(q.device).data_ptr(), stream_ptr()), "latent_prefill")
         return out
     check(lib().ttb_latent_attention_any(q.data_ptr(), s * _pitch(q), _pitch(q), dim + rot, kn.data_ptr(), sk * _pitch(kn), _pitch(kn), dim, kr_ptr, buf.shape[1] * width, width,
-                                         v.data_ptr(), sk * _pitch(v), _pitch(v), vdim, out.data_ptr(), None, _p(gate), 0 if gate is None else _pitch(gate), b, s, sk, heads, dim, rot, vdim,
+                                         v.data_ptr(), sk * _pitch(v), _pitch(v), vdim, out.data_ptr(), None, _p(gate), 0 if gate is None else _pitch(gate), b, s, sk, heads, 1, dim, rot, vdim,
                                          0, 0, None, slot0, _p(bounds.lo), bounds.lo_row, bounds.lo_query, _p(bounds.hi), bounds.hi_row, bounds.hi_query, float(scale), _wide(q),
                                          stream_ptr()), "latent_attention_any (prefill)")
     return out
@@ -147,7 +147,7 @@ def decode(q_lat: torch.Tensor, buf: torch.Tensor, *, rank: int, rot: int, scale
     ml = torch.empty(1, b, heads, 2, dtype=torch.float32, device=q_lat.device)
     c = buf.data_ptr()
     check(lib().ttb_latent_attention_any(q_lat.data_ptr(), heads * width, 0, width, c, slots * width, width, 0, c + rank * buf.element_size(), slots * width, width, c, slots * width, width, 0,
-                                         o.data_ptr(), ml.data_ptr(), None, 0, b, 1, slots, heads, rank, rot, rank, 1, 1, _p(slot), int(slot_host), _p(bounds.lo), bounds.lo_row, 0,
+                                         o.data_ptr(), ml.data_ptr(), None, 0, b, 1, slots, heads, heads, rank, rot, rank, 1, 1, _p(slot), int(slot_host), _p(bounds.lo), bounds.lo_row, 0,
                                          _p(bounds.hi), bounds.hi_row, 0, float(scale), _wide(q_lat), stream_ptr()), "latent_attention_any (decode)")
     return o, ml
 
