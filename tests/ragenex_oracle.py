@@ -186,7 +186,7 @@ def weights(cfg, seed=0, sharp=2.0):
         z = rng.normal(0.0, 1.0, shape)
         last = name.split(".")[-1]
         if ".hc" in name:
-            z = {"in": 1.0 / S + 0.3 * z, "out": 1.0 + 0.4 * z, "mix": np.eye(S) * 0.9 + 0.1 * z if z.ndim == 2 else z}[last]
+            z = {"in": 1.0 / S + 0.3 * z, "out": 0.6 + 0.3 * z, "mix": np.eye(S) * 0.9 + 0.1 * z if z.ndim == 2 else z}[last]
         elif z.ndim == 1:
             z = 1.0 + 0.2 * z
             z = z * (sharp if name.endswith("q.norm") else 1.0)

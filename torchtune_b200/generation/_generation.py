@@ -110,6 +110,9 @@ def generate(
     mask_width = model.decoder_max_cache_seq_len if incremental else total_len
 
     real = prompt != pad_id
+    limit = getattr(model, "position_limit", None)
+    if limit is not None and int(real.sum(1).max()) + max_generated_tokens - 1 > limit:
+        raise ValueError(f"{int(real.sum(1).max())} prompt tokens and {max_generated_tokens} generated ones are more than the model's {limit} positions")
     layout = RowLayout(real) if incremental and getattr(model, "span_masks", False) else None
     if layout is not None:
         masks = input_pos = None

@@ -120,6 +120,7 @@ class BatchDecoder:
         self.model, self.device, self.dtype, self.max_tokens = model, device, dtype, int(max_tokens)
         self.layout: Optional[RowLayout] = None
         self.used = 0
+        self.lengths: List[int] = []  # tokens of each live row
         self._capacity = (0, 0)
         self._graphs = graphs and device.type == "cuda"
         self._graph: Optional[DecodeGraph] = None
@@ -146,17 +147,25 @@ class BatchDecoder:
         longest, shortest = max(lengths), min(lengths)
         if shortest < 1:
             raise ValueError("a row starts with at least one token")
+        self._check_positions(longest)
         # a row may go on alone until it holds every token of the budget: that many slots behind the padding of the shortest one
         self._reserve(len(prompts), longest + max(self.max_tokens - shortest, 0))
         tokens = torch.tensor([[0] * (longest - n) + p for p, n in zip(prompts, lengths)], device=self.device)
         real = torch.arange(longest)[None, :] >= torch.tensor([longest - n for n in lengths])[:, None]
-        self.layout, self.used = RowLayout(real.to(self.device)), 0
+        self.layout, self.used, self.lengths = RowLayout(real.to(self.device)), 0, lengths
         return self._run(tokens)
+
+    def _check_positions(self, length: int) -> None:
+        limit = getattr(self.model, "position_limit", None)
+        if limit is not None and length > limit:
+            raise ValueError(f"a row of {length} tokens is longer than the model's {limit} positions")
 
     def advance(self, tokens: List[int]) -> torch.Tensor:
         """Hidden states ``[b, 1, d]`` of one more token per live row."""
         if len(tokens) != self.rows or not tokens:
             raise ValueError(f"{len(tokens)} tokens for {self.rows} rows")
+        self._check_positions(max(self.lengths) + 1)
+        self.lengths = [n + 1 for n in self.lengths]
         step = torch.tensor(tokens, device=self.device)[:, None]
         if not self._graphs:
             return self._run(step)
@@ -180,12 +189,13 @@ class BatchDecoder:
         gone = set(rows)
         kept = [i for i in range(self.rows) if i not in gone]
         if not kept:
-            self.layout, self.used, self._graph = None, 0, None
+            self.layout, self.used, self.lengths, self._graph = None, 0, [], None
             self.model.reset_caches()
             return
         if len(kept) == self.rows:
             return
         self._graph = None
+        self.lengths = [self.lengths[i] for i in kept]
         for layer in self.model.layers:
             cache = layer.attn.kv_cache
             if cache is not None:

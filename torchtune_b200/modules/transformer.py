@@ -418,6 +418,11 @@ class TransformerDecoder(nn.Module):
             return input_embeds.float() + self.pos_embeddings(pos).float()
         return ops.embed_positions(tokens, pos, self.tok_embeddings.weight, self.pos_embeddings.weight)
 
+    @property
+    def position_limit(self) -> Optional[int]:
+        """Longest sequence the position embeddings reach; ``None`` without a table."""
+        return None if self.pos_embeddings is None else self.pos_embeddings.num_embeddings
+
     def unembed_normed(self, h: torch.Tensor) -> torch.Tensor:
         if self.wide_logits and type(self.output).__name__ == "Linear" and self.output.bias is None:
             return self._cap(ops.linear_wide(h, self.output.weight))
