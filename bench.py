@@ -587,7 +587,8 @@ def run_ours_sharded(args) -> dict:
     return out if rank == 0 else {}
 
 
-# Serving comparison (``--serve``): a Begapel decoder and the closest other decoder of equal width, heads, feed-forward and depth.
+# Serving comparison (``--serve``): a Begapel or Ragenex decoder (``--serve-model``) and the closest other decoders of equal width, heads,
+# feed-forward and depth.
 SERVE_SIZES = {
     "1b": dict(width=2048, heads=16, ff=8192, layers=12, vocab=65_536),
     "3b": dict(width=4096, heads=32, ff=14_336, layers=8, vocab=65_536),
@@ -597,7 +598,8 @@ SERVE_ROT, SERVE_RANK, SERVE_DIM = 64, 512, 128
 
 def run_serve(args) -> dict:
     """Prefill and decode throughput through the generation path, random weights: ``--serve 1b | 3b``.  Begapel layers (every fourth one
-    without latents of its own) against llama3_1 layers with a quarter as many key heads."""
+    without latents of its own) against llama3_1 layers with a quarter as many key heads; or Ragenex layers (lightning and attention layers in
+    turn, four residual streams) against both."""
     import torch
 
     from torchtune_b200 import training
@@ -617,11 +619,20 @@ def run_serve(args) -> dict:
 
     cfg = {"architecture": "Begapel", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 30.0,
            "layers": [{"type": "latent_attention", "mixer": mixer(i), "mlp": {"kind": "dense", "ff": z["ff"]}} for i in range(z["layers"])]}
+    glu = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    lightning = {"type": "lightning", "mixer": {"heads": z["heads"], "dim": SERVE_DIM, "vdim": SERVE_DIM, "decay": [1.0 - 2.0 ** -(1 + 10 * h / z["heads"]) for h in range(z["heads"])]}, "mlp": glu}
+    attention = {"type": "attention", "mixer": {"heads": z["heads"], "kv_heads": z["heads"] // 4, "dim": SERVE_DIM, "vdim": SERVE_DIM, "scale": SERVE_DIM**-0.5,
+                                                "q_temp": {"coef": 0.1, "every": 1024}}, "mlp": glu}
+    ragenex_cfg = {"architecture": "Ragenex", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-6}, "streams": 4, "max_positions": 16384,
+                   "layers": [(lightning, attention)[i % 2] for i in range(z["layers"])]}
     builders = {
+        "ragenex": lambda: build_from_config(ragenex_cfg),
         "begapel": lambda: build_from_config(cfg, max_seq_len=16384),
         "llama3_1": lambda: llama3_1(vocab_size=z["vocab"], num_layers=z["layers"], num_heads=z["heads"], num_kv_heads=z["heads"] // 4, embed_dim=z["width"], max_seq_len=16384,
                                      intermediate_dim=z["ff"]),
     }
+    if args.serve_model == "begapel":
+        del builders["ragenex"]
 
     def timed(fn, n):
         for i in range(max(3, args.warmup)):
@@ -686,9 +697,9 @@ def run_serve(args) -> dict:
             torch.cuda.empty_cache()
     clocks = sampler.stop()
     check_device_errors()
-    return {"metric": "serving_tokens_per_second", "value": results["begapel"]["decode_b16_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
+    return {"metric": "serving_tokens_per_second", "value": results[args.serve_model]["decode_b16_tokens_per_s"], "unit": "tokens/s", "n_gpus": 1, "steps": args.steps, "warmup": args.warmup,
             "higher_is_better": True, "vs_baseline": None, "dtype": "bf16", "data": "synthetic tokens, random-init weights", "impl": "ours",
-            "config": {"serve": args.serve, **z, "prompt_tokens": prompt, "decode_context": context, "l2": "weights and caches larger than L2"}, "results": results, "clocks": clocks,
+            "config": {"serve": args.serve, "model": args.serve_model, **z, "prompt_tokens": prompt, "decode_context": context, "l2": "weights and caches larger than L2"}, "results": results, "clocks": clocks,
             "gpu_launches": int(lib().ttb_launch_count() - launches0)}
 
 
@@ -721,7 +732,8 @@ def main() -> None:
     ap.add_argument("--ref-compile", action="store_true", help="with --impl reference: the reference's `compile: True` path (informational; the default arm stays on the stock eager path)")
     ap.add_argument("--fp8-recipe", choices=["tensorwise", "blockwise"], default="tensorwise", help="with --fp8: one scale per tensor, or MX block scales (32 values per scale)")
     ap.add_argument("--fp8", action="store_true", help="variant: fp8 decoder linears (the headline number is always bf16)")
-    ap.add_argument("--serve", choices=sorted(SERVE_SIZES), default=None, help="prefill and decode throughput of Begapel layers beside llama3_1 layers of equal size, instead of the training step")
+    ap.add_argument("--serve", choices=sorted(SERVE_SIZES), default=None, help="prefill and decode throughput of a serving model beside other models of equal size, instead of the training step")
+    ap.add_argument("--serve-model", choices=["begapel", "ragenex"], default="begapel", help="with --serve: the model to measure; begapel beside llama3_1, ragenex beside both")
     args = ap.parse_args()
     rank, world, _ = dist_env()
     if args.gpus > 1 and world == 1:

@@ -383,7 +383,7 @@ MODELS = {
     "plain": lambda: oracle.config([oracle.attention_layer(), oracle.lightning_layer(), oracle.attention_layer(heads=4, kv_heads=4, dim=40, vdim=16, ff=None)]),
     "looped": lambda: oracle.config([oracle.lightning_layer(ff=None), oracle.attention_layer(heads=5, kv_heads=1, dim=64, vdim=72, coef=0.3, every=17), oracle.lightning_layer(decay=(0.8, 0.99), dim=40, vdim=16),
                                      oracle.attention_layer()], loop=(0, 3, 2), streams=4, width=136, eps=3e-2),
-    "odd": lambda: oracle.config([oracle.lightning_layer(decay=(0.9,), dim=5, vdim=7, ff=35), oracle.attention_layer(heads=3, kv_heads=3, dim=11, vdim=9, every=1, ff=22)], width=51, vocab=67, streams=1,
+    "odd": lambda: oracle.config([oracle.lightning_layer(decay=(0.9, 0.98, 0.7), dim=13, vdim=11, ff=35), oracle.attention_layer(heads=3, kv_heads=3, dim=11, vdim=9, every=1, ff=22)], width=51, vocab=67, streams=1,
                                  loop=(1, 2, 2), eps=1e-2),
     "large": lambda: oracle.config([oracle.attention_layer(heads=36, kv_heads=2, dim=128, vdim=128, ff=64), oracle.lightning_layer(decay=(0.97, 0.9999), dim=128, vdim=128, ff=64)], width=72, streams=2),
 }

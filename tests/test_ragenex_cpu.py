@@ -450,6 +450,9 @@ def test_checkpoint_round_trip(tmp_path):
     assert torch.equal(again(torch.tensor([s])), model(torch.tensor([s])))
     with pytest.raises(ValueError, match="unexpected tensor"):
         ragenex_hf_to_tune({"l0.mix.z": torch.zeros(1)})
+    extra = {**w, "l0.norm2": w["l0.norm1"], "l0.hc2.in": w["l0.hc1.in"]}  # layer 0 has no feed-forward block
+    more = load_pretrained(oracle.save(tmp_path / "b", cfg, extra), dtype=torch.float32, device=CPU)
+    assert torch.equal(more(torch.tensor([s])), model(torch.tensor([s])))
 
 
 def test_configuration_is_checked(tmp_path):

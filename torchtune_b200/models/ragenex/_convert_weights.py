@@ -3,7 +3,7 @@ stacked along the rows, mixing weights ``[from, to]``)."""
 from __future__ import annotations
 
 import re
-from typing import Dict
+from typing import Any, Dict, Mapping, Optional
 
 import torch
 
@@ -35,10 +35,18 @@ _LAYER_BACK = {v: k for k, v in _LAYER.items()}
 _TOP_BACK = {v: k for k, v in _TOP.items()}
 
 
-def ragenex_hf_to_tune(state_dict: Dict[str, torch.Tensor]) -> Dict[str, torch.Tensor]:
+_FEED_FORWARD = ("norm2", "ls2", "hc2.", "mlp.")
+
+
+def ragenex_hf_to_tune(state_dict: Dict[str, torch.Tensor], config: Optional[Mapping[str, Any]] = None) -> Dict[str, torch.Tensor]:
+    """With the model's ``config``, tensors around a feed-forward block that a layer does not have are left out."""
+    layers = (config or {}).get("layers") or []
+    bare = {i for i, layer in enumerate(layers) if layer.get("mlp") is None}
     out = {}
     for key, value in state_dict.items():
         m = re.fullmatch(r"l(\d+)\.(.+)", key)
+        if m and int(m.group(1)) in bare and m.group(2).startswith(_FEED_FORWARD):
+            continue
         if m and m.group(2) in _LAYER:
             out[f"layers.{m.group(1)}.{_LAYER[m.group(2)]}"] = value
         elif key in _TOP:
@@ -65,7 +73,7 @@ def _register() -> None:
     from ...training.checkpointing._codecs import register_hf_codec
     from ...training.checkpointing._utils import ModelType
 
-    register_hf_codec(ModelType.RAGENEX, lambda sd, cfg: ragenex_hf_to_tune(sd), lambda sd, cfg: ragenex_tune_to_hf(sd))
+    register_hf_codec(ModelType.RAGENEX, lambda sd, cfg: ragenex_hf_to_tune(sd, cfg), lambda sd, cfg: ragenex_tune_to_hf(sd))
 
 
 _register()

@@ -47,6 +47,27 @@ __device__ __forceinline__ uint4 pack_bf16x8(const float (&f)[8]) {
   return u;
 }
 
+// Lanes 4m ... 4m + 3 hold four 16-byte pieces each; piece j of lane 4m + i becomes piece i of lane 4m + j.  A warp whose lanes hold rows so
+// turns 16-byte accesses to 32 rows into 64-byte accesses to eight.  All lanes take part.
+__device__ __forceinline__ void transpose_quads(uint4 (&v)[4]) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int bit = 1; bit <= 2; bit <<= 1) {
+    const bool upper = lane & bit;
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+      const int a = bit == 1 ? 2 * k : k, b = a + bit;
+      uint4 t = upper ? v[a] : v[b];
+      t.x = __shfl_xor_sync(0xffffffffu, t.x, bit);
+      t.y = __shfl_xor_sync(0xffffffffu, t.y, bit);
+      t.z = __shfl_xor_sync(0xffffffffu, t.z, bit);
+      t.w = __shfl_xor_sync(0xffffffffu, t.w, bit);
+      if (upper) v[a] = t;
+      else v[b] = t;
+    }
+  }
+}
+
 // 1 / (1 + e^-z): the fast exponential where the result is rounded to bf16 anyway, the full-precision one for fp32 tensors
 template <typename T>
 __device__ __forceinline__ float logistic(float z) {

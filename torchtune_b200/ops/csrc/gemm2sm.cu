@@ -41,6 +41,9 @@ static constexpr int kStagesSwiglu = 5;
 static constexpr int kSmemBytesSwiglu = kStagesSwiglu * kStageBytes + 1024 + 2 * kEpiBytes + 1024;
 static_assert(kSmemBytesSwiglu <= 232448, "shared memory budget of one CTA");
 
+// What the epilogue of the gate / up form computes: silu(g)·u, or g·sigmoid(alpha·g)·(u + 1) with both pre-activations clamped.
+enum Gate { kNoGate = 0, kSwiglu = 1, kClampedGate = 2 };
+
 struct Params {
   int M, N, K;
   int K2;  // > 0: a second operand pair (tmA2, tmB2) with K2 contraction columns extends the main loop (LoRA: one accumulator)
@@ -54,7 +57,7 @@ struct Params {
   int tma_store;
   int group_m;  // pair-tiles in m per scheduling group
   int tile_mult;  // 1, or an odd multiplier coprime to the tile count: tile t is replaced by (t · tile_mult) mod tiles (debug aid)
-  float glu_limit, glu_alpha;  // SWIGLU form, limit > 0: g·sigmoid(alpha·g)·(u + 1) with both pre-activations clamped, instead of silu(g)·u
+  float glu_limit, glu_alpha;  // clamped gate
   int save_gate_up;  // SWIGLU form: also store the two pre-activations (the backward pass needs them)
   int* err;
 };
@@ -122,11 +125,12 @@ __device__ __forceinline__ void tile_coords(int t, int num_m, int num_n, int gro
 // of the same 128 hidden units, in both CTAs' tensor memory.  The epilogue writes h = silu(gate) · up ([M, N], N = hidden width; tmC) and,
 // when the backward pass will need them, gate and up as well (tmG, tmU).  The separate SwiGLU kernel and its re-read of both
 // pre-activations disappear; in a gradient-free forward pass the pre-activations never reach HBM at all.
-template <bool A_MN, bool B_MN, bool SWIGLU>
+template <bool A_MN, bool B_MN, int GLU>
 __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(kThreads, 1)
 gemm2sm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB, const __grid_constant__ CUtensorMap tmC,
                const __grid_constant__ CUtensorMap tmB2, const __grid_constant__ CUtensorMap tmG, const __grid_constant__ CUtensorMap tmU,
                const __grid_constant__ CUtensorMap tmA2, Params p) {
+  constexpr bool SWIGLU = GLU != kNoGate;
   constexpr int kNS = SWIGLU ? kStagesSwiglu : kStages;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -321,9 +325,9 @@ gemm2sm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
                 // round the pre-activations to bf16 first: the unfused path computes SwiGLU from the stored bf16 values
                 g[i] = __bfloat162float(__float2bfloat16_rn(__uint_as_float(rg[j * 8 + i])));
                 u[i] = __bfloat162float(__float2bfloat16_rn(__uint_as_float(ru[j * 8 + i])));
-                if (p.glu_limit > 0.f) {
+                if constexpr (GLU == kClampedGate) {
                   const float gc = fminf(g[i], p.glu_limit), uc = fminf(fmaxf(u[i], -p.glu_limit), p.glu_limit);
-                  o[i] = gc / (1.f + __expf(-p.glu_alpha * gc)) * (uc + 1.f);
+                  o[i] = __fdividef(gc, 1.f + __expf(-p.glu_alpha * gc)) * (uc + 1.f);
                 } else {
                   o[i] = g[i] / (1.f + __expf(-g[i])) * u[i];
                 }
@@ -502,9 +506,10 @@ static int shuffle_multiplier(int num_tiles) {
   return m;
 }
 
-template <bool A_MN, bool B_MN, bool SWIGLU>
+template <bool A_MN, bool B_MN, int GLU>
 static int launch(const void* A, const void* B, const void* B2, void* G, void* U, const Params& p, long long lda, long long ldb, cudaStream_t stream,
                   const void* A2 = nullptr, long long lda2 = 0, long long ldb2 = 0) {
+  constexpr bool SWIGLU = GLU != kNoGate;
   CUtensorMap tmA, tmB, tmB2, tmC, tmG, tmU, tmA2;
   memset(&tmA2, 0, sizeof(tmA2));
   memset(&tmB2, 0, sizeof(tmB2));
@@ -545,7 +550,7 @@ static int launch(const void* A, const void* B, const void* B2, void* G, void* U
   } else {
     q.tma_store = (!p.accumulate && (reinterpret_cast<uintptr_t>(p.C) & 15) == 0 && map_c(&tmC, p.C) == kOk) ? 1 : 0;
   }
-  auto kern = gemm2sm_kernel<A_MN, B_MN, SWIGLU>;
+  auto kern = gemm2sm_kernel<A_MN, B_MN, GLU>;
   constexpr int smem = SWIGLU ? kSmemBytesSwiglu : kSmemBytes;
   static bool attr_set = false;
   if (!attr_set) {
@@ -587,8 +592,8 @@ extern "C" int ttb_gemm_bf16_2sm(const void* A, const void* B, void* C, int M, i
   p.residual = nullptr, p.ldr = 0;
   p.group_m = g2::group_setting();
   auto s = static_cast<cudaStream_t>(stream);
-  if (a_mn) return b_mn ? g2::launch<true, true, false>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s) : g2::launch<true, false, false>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s);
-  return b_mn ? g2::launch<false, true, false>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s) : g2::launch<false, false, false>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s);
+  if (a_mn) return b_mn ? g2::launch<true, true, g2::kNoGate>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s) : g2::launch<true, false, g2::kNoGate>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s);
+  return b_mn ? g2::launch<false, true, g2::kNoGate>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s) : g2::launch<false, false, g2::kNoGate>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, s);
 }
 
 // C[M,N] = alpha · (A·op(B) + A2·op(B2)) (+ bias) on CTA pairs: the second pair's k-blocks (K2 columns, zero-filled up to a multiple of
@@ -606,8 +611,8 @@ extern "C" int ttb_gemm_bf16_dual_2sm(const void* A, const void* B, const void* 
   p.accumulate = 0, p.tma_store = 0, p.save_gate_up = 0, p.tile_mult = 1, p.err = err;
   p.group_m = g2::group_setting();
   auto s = static_cast<cudaStream_t>(stream);
-  return b_mn ? g2::launch<false, true, false>(A, B, B2, nullptr, nullptr, p, lda, ldb, s, A2, lda2, ldb2)
-              : g2::launch<false, false, false>(A, B, B2, nullptr, nullptr, p, lda, ldb, s, A2, lda2, ldb2);
+  return b_mn ? g2::launch<false, true, g2::kNoGate>(A, B, B2, nullptr, nullptr, p, lda, ldb, s, A2, lda2, ldb2)
+              : g2::launch<false, false, g2::kNoGate>(A, B, B2, nullptr, nullptr, p, lda, ldb, s, A2, lda2, ldb2);
 }
 
 // Gated MLP up-projection with the activation in the epilogue: H[M, N] = silu(X · W1ᵀ) ⊙ (X · W3ᵀ) with X [M, K], W1 and W3 [N, K]
@@ -626,7 +631,9 @@ extern "C" int ttb_gemm_swiglu_bf16_2sm(const void* X, const void* W1, const voi
   p.accumulate = 0, p.tma_store = 1, p.save_gate_up = 0, p.tile_mult = 1, p.err = err, p.K2 = 0;
   p.glu_limit = glu_limit, p.glu_alpha = glu_alpha;
   p.group_m = g2::group_setting();
-  return g2::launch<false, false, true>(X, W1, W3, gate_out, up_out, p, lda, ldb, static_cast<cudaStream_t>(stream));
+  auto s = static_cast<cudaStream_t>(stream);
+  return glu_limit > 0.f ? g2::launch<false, false, g2::kClampedGate>(X, W1, W3, gate_out, up_out, p, lda, ldb, s)
+                         : g2::launch<false, false, g2::kSwiglu>(X, W1, W3, gate_out, up_out, p, lda, ldb, s);
 }
 
 
@@ -643,5 +650,5 @@ extern "C" int ttb_gemm_bf16_2sm_residual(const void* A, const void* B, void* C,
   p.residual = static_cast<const __nv_bfloat16*>(R), p.ldr = ldr;
   p.accumulate = 0, p.tma_store = 0, p.save_gate_up = 0, p.tile_mult = 1, p.err = err;
   p.group_m = g2::group_setting();
-  return g2::launch<false, false, false>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, static_cast<cudaStream_t>(stream));
+  return g2::launch<false, false, g2::kNoGate>(A, B, nullptr, nullptr, nullptr, p, lda, ldb, static_cast<cudaStream_t>(stream));
 }

@@ -157,8 +157,9 @@ struct ChunkParams {
 };
 
 static constexpr int kChunkThreads = 384;
+static constexpr int kRunThreads = 640;
 static constexpr int kTile = 2 * kPanelBytes;  // 128 rows x 128 columns
-static constexpr int kRunSmem = 7 * kTile + 1024 + 32 * 8 + 132 * 4;
+static constexpr int kRunSmem = 7 * kTile + 1024 + 32 * 8 + 260 * 4;
 static constexpr int kRunStateSmem = 6 * kTile + 1024 + 32 * 8 + 132 * 4;
 static_assert(kRunSmem <= 227 * 1024 && kRunStateSmem <= 227 * 1024, "shared memory of one CTA");
 
@@ -185,6 +186,36 @@ __device__ __forceinline__ void scale_panel_row(const uint8_t* v, uint8_t* hi, u
     split2(f[6] * w, f[7] * w, a.w, b.w);
     *reinterpret_cast<uint4*>(hi + at) = a;
     *reinterpret_cast<uint4*>(lo + at) = b;
+  }
+}
+
+// 32 columns of a state row per lane (rows row0 + lane) <-> the state in memory [dk, dv], 64 bytes of a row at a time.
+__device__ __forceinline__ void store_state_piece(float* state, const uint32_t (&v)[32], int row0, int col0, int dk, int dv) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int g = 0; g < 2; ++g) {
+    uint4 q[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) q[j] = make_uint4(v[g * 16 + j * 4], v[g * 16 + j * 4 + 1], v[g * 16 + j * 4 + 2], v[g * 16 + j * 4 + 3]);
+    transpose_quads(q);
+    const int row = row0 + (lane & ~3), col = col0 + g * 16 + (lane & 3) * 4;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (row + j < dk && col < dv) *reinterpret_cast<uint4*>(state + static_cast<long long>(row + j) * dv + col) = q[j];
+  }
+}
+__device__ __forceinline__ void load_state_piece(const float* state, uint32_t (&v)[32], int row0, int col0, int dk, int dv) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int g = 0; g < 2; ++g) {
+    uint4 q[4];
+    const int row = row0 + (lane & ~3), col = col0 + g * 16 + (lane & 3) * 4;
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      q[j] = state != nullptr && row + j < dk && col < dv ? *reinterpret_cast<const uint4*>(state + static_cast<long long>(row + j) * dv + col) : make_uint4(0u, 0u, 0u, 0u);
+    transpose_quads(q);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[g * 16 + j * 4] = q[j].x, v[g * 16 + j * 4 + 1] = q[j].y, v[g * 16 + j * 4 + 2] = q[j].z, v[g * 16 + j * 4 + 3] = q[j].w;
   }
 }
 
@@ -284,18 +315,13 @@ lightning_run_state_kernel(const __grid_constant__ CUtensorMap tmK, const __grid
       if (ok && !*abort_flag) ok = mbar_wait(done, 0);
       if (ok && !*abort_flag) {
         tc_fence_after();
-        float* dst = p.run_state + (((static_cast<long long>(bi) * p.heads + h) * p.runs + run) * p.dk + row) * p.dv;
+        float* dst = p.run_state + ((static_cast<long long>(bi) * p.heads + h) * p.runs + run) * p.dk * p.dv;
 #pragma unroll 1
         for (int ch = 0; ch < p.v_panels * 2; ++ch) {
           uint32_t v[32];
           tmem_ld_32x32(tH + (static_cast<uint32_t>((warp & 3) * 32) << 16) + ch * 32, v);
           tmem_ld_wait();
-          if (row < p.dk) {
-#pragma unroll
-            for (int i = 0; i < 32; i += 4)
-              if (ch * 32 + i < p.dv)
-                *reinterpret_cast<float4*>(dst + ch * 32 + i) = make_float4(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), __uint_as_float(v[i + 2]), __uint_as_float(v[i + 3]));
-          }
+          store_state_piece(dst, v, (warp & 3) * 32, ch * 32, p.dk, p.dv);
         }
       }
     }
@@ -318,19 +344,27 @@ __global__ void __launch_bounds__(256) lightning_scan_kernel(float* __restrict__
   float cur[4] = {0.f, 0.f, 0.f, 0.f};
   if (state != nullptr) load4(state + row * n + i, cur);
   float* w = work + row * runs * n + i;
-  for (int r = 0; r < runs; ++r, w += n) {
-    float add[4] = {0.f, 0.f, 0.f, 0.f};
-    if (r + 1 < runs) load4(w, add);
-    store4(w, cur);
+  for (int r0 = 0; r0 < runs; r0 += 8) {
+    float add[8][4];
 #pragma unroll
-    for (int j = 0; j < 4; ++j) cur[j] = by * cur[j] + add[j];
+    for (int r = 0; r < 8; ++r) {  // the loads of eight runs are in flight together
+      add[r][0] = add[r][1] = add[r][2] = add[r][3] = 0.f;
+      if (r0 + r + 1 < runs) load4(w + (r0 + r) * n, add[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < 8; ++r) {
+      if (r0 + r >= runs) break;
+      store4(w + (r0 + r) * n, cur);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) cur[j] = by * cur[j] + add[r][j];
+    }
   }
 }
 
-// One run of one head.  Warp 0 loads, warp 1 issues the products, warps 4 - 7 turn scores into weights and write the output, warps 8 - 11
-// keep the state: once per chunk its two bf16 parts go to shared memory for the product with the queries, it is decayed in place, and the
+// One run of one head.  Warp 0 loads, warp 1 issues the products, warps 4 - 11 turn scores into weights and write the output, warps 12 - 19
+// keep the state (each group of four warps has all rows and half of the columns): once per chunk its two bf16 parts go to shared memory for the product with the queries, it is decayed in place, and the
 // scaled values (also in two parts, in the same shared memory) are multiplied onto it.
-__global__ void __launch_bounds__(kChunkThreads, 1)
+__global__ void __launch_bounds__(kRunThreads, 1)
 lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const ChunkParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
@@ -355,7 +389,7 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   uint64_t* o_free = bars + 15;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 16);
   volatile int* abort_flag = reinterpret_cast<volatile int*>(tmem_slot + 1);
-  float* pw = reinterpret_cast<float*>(bars + 32);
+  float* pw = reinterpret_cast<float*>(bars + 32) + kBlk;  // powers of the decay: pw[-128 ... -1] = 0, pw[0 ... 128]
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int run = blockIdx.x, h = blockIdx.y, bi = blockIdx.z;
   const int tok0 = run * p.run_chunks * kBlk;
@@ -371,17 +405,18 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       mbar_init(&kv_empty[i], 1);
     }
     mbar_init(s_full, 1);
-    mbar_init(p_full, 4);
-    mbar_init(st_full, 4);
+    mbar_init(p_full, 8);
+    mbar_init(st_full, 8);
     mbar_init(t_done, 1);
-    mbar_init(vs_full, 4);
+    mbar_init(vs_full, 8);
     mbar_init(h_done, 1);
     mbar_init(o_full, 1);
-    mbar_init(o_free, 4);
+    mbar_init(o_free, 8);
     *abort_flag = 0;
     fence_mbar_init();
   }
   if (threadIdx.x < kBlk + 1) pw[threadIdx.x] = p.powers[h * (kBlk + 1) + threadIdx.x];
+  else if (threadIdx.x < 2 * kBlk + 1) pw[kBlk - static_cast<int>(threadIdx.x)] = 0.f;
   if (warp == 2) {
     tmem_alloc(tmem_slot, 512);
     tmem_relinquish();
@@ -451,7 +486,7 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       tc_fence_after();
       if (ok && elect_one()) {
 #pragma unroll
-        for (int i = 0; i < kBlk / 16; ++i) umma_f16_ts(tO, tS + i * 8, desc_mnmajor(aV, i), idesc_o, i != 0);
+        for (int i = 0; i < kBlk / 16; ++i) umma_f16_ts(tO, tS + (i >> 2) * 64 + (i & 3) * 8, desc_mnmajor(aV, i), idesc_o, i != 0);
         umma_commit(o_full);
       }
       __syncwarp();
@@ -469,9 +504,9 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       __syncwarp();
     }
     if (!ok) fail(abort_flag, p.err, 253);
-  } else if (warp >= 4 && warp < 8) {
-    // ---------------------------------------------------------------- weights and output, one query row per thread
-    const int quarter = warp & 3, r = quarter * 32 + lane;
+  } else if (warp >= 4 && warp < 12) {
+    // ---------------------------------------------------------------- weights and output: one query row and 64 keys / one value panel per thread
+    const int quarter = warp & 3, r = quarter * 32 + lane, part = (warp - 4) >> 2;
     const uint32_t lane_sel = static_cast<uint32_t>(quarter * 32) << 16;
     bool ok = true;
     for (int c = 0; c < n && ok && !*abort_flag; ++c) {
@@ -480,21 +515,24 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       ok = mbar_wait(s_full, ph);
       if (!ok) break;
       tc_fence_after();
+      const uint32_t scores = tS + lane_sel + part * 64;
+      uint32_t pk[32];
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
-        uint32_t sv[2][32], pk[32];
-        tmem_ld_32x32(tS + lane_sel + half * 64, sv[0]);
-        tmem_ld_32x32(tS + lane_sel + half * 64 + 32, sv[1]);
+        uint32_t sv[32];
+        tmem_ld_32x32(scores + half * 32, sv);
         tmem_ld_wait();
+        const int j0 = part * 64 + half * 32;
+        const float* w = pw + r - j0;
+        if (lo > j0) {
 #pragma unroll
-        for (int i = 0; i < 64; i += 2) {
-          const int j = half * 64 + i;
-          const float a = j <= r && j >= lo ? __uint_as_float(sv[i >> 5][i & 31]) * pw[r - j] : 0.f;
-          const float b = j + 1 <= r && j + 1 >= lo ? __uint_as_float(sv[i >> 5][(i & 31) + 1]) * pw[r - j - 1] : 0.f;
-          pk[i >> 1] = pack_bf16x2(a, b);
+          for (int i = 0; i < 32; ++i)
+            if (j0 + i < lo) sv[i] = 0u;
         }
-        tmem_st_32x32(tS + lane_sel + half * 32, pk);  // over scores that have been read
+#pragma unroll
+        for (int i = 0; i < 32; i += 2) pk[half * 16 + (i >> 1)] = pack_bf16x2(__uint_as_float(sv[i]) * w[-i], __uint_as_float(sv[i + 1]) * w[-i - 1]);
       }
+      tmem_st_32x32(scores, pk);  // over this group's own scores
       tmem_st_wait();
       tc_fence_before();
       __syncwarp();
@@ -503,35 +541,38 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       if (!ok) break;
       tc_fence_after();
       const float by = pw[r + 1];
-      const bool valid = tok + r < p.s;
-      bf16* dst = p.o + ((static_cast<long long>(bi) * p.s + tok + r) * p.heads + h) * p.dv;
+      bf16* dst = p.o + ((static_cast<long long>(bi) * p.s + tok) * p.heads + h) * p.dv;
 #pragma unroll 1
-      for (int ch = 0; ch < p.v_panels * 2; ++ch) {
+      for (int ch = part * 2; ch < part * 2 + 2 && part < p.v_panels; ++ch) {
         uint32_t t[32], o[32];
         tmem_ld_32x32(tT + lane_sel + ch * 32, t);
         tmem_ld_32x32(tO + lane_sel + ch * 32, o);
         tmem_ld_wait();
-        if (!valid) continue;
+        uint4 q[4];
 #pragma unroll
         for (int g = 0; g < 4; ++g) {
-          const int col = ch * 32 + g * 8;
-          if (col >= p.dv) continue;  // dv is a multiple of 8
           float f[8];
 #pragma unroll
           for (int i = 0; i < 8; ++i) f[i] = by * __uint_as_float(t[g * 8 + i]) + __uint_as_float(o[g * 8 + i]);
-          *reinterpret_cast<uint4*>(dst + col) = pack_bf16x8(f);
+          q[g] = pack_bf16x8(f);
         }
+        transpose_quads(q);
+        const int row = quarter * 32 + (lane & ~3), col = ch * 32 + (lane & 3) * 8;  // dv is a multiple of 8
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          if (tok + row + j < p.s && col < p.dv) *reinterpret_cast<uint4*>(dst + static_cast<long long>(row + j) * p.heads * p.dv + col) = q[j];
       }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(o_free);
     }
     if (!ok) fail(abort_flag, p.err, 254);
-  } else if (warp >= 8) {
-    // ---------------------------------------------------------------- state: one state row, later one token's values, per thread
-    const int quarter = warp & 3, r = quarter * 32 + lane;
+  } else if (warp >= 12) {
+    // ---------------------------------------------------------------- state: one panel of one state row, later of one token's values, per thread
+    const int quarter = warp & 3, r = quarter * 32 + lane, part = (warp - 12) >> 2;
+    const int first_ch = part * 2, last_ch = part < p.v_panels ? first_ch + 2 : first_ch;  // 32-column pieces
     const uint32_t lane_sel = static_cast<uint32_t>(quarter * 32) << 16;
-    const float* begin = p.begin != nullptr && r < p.dk ? p.begin + (((static_cast<long long>(bi) * p.heads + h) * p.runs + run) * p.dk + r) * p.dv : nullptr;
+    const float* begin = p.begin != nullptr ? p.begin + ((static_cast<long long>(bi) * p.heads + h) * p.runs + run) * p.dk * p.dv : nullptr;
     bool ok = true;
     for (int c = 0; c < n && ok && !*abort_flag; ++c) {
       const uint32_t ph = c & 1;
@@ -543,19 +584,13 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       }
       const float by = pw[count];
 #pragma unroll 1
-      for (int ch = 0; ch < p.v_panels * 2; ++ch) {
+      for (int ch = first_ch; ch < last_ch; ++ch) {
         uint32_t v[32];
         if (c > 0) {
           tmem_ld_32x32(tH + lane_sel + ch * 32, v);
           tmem_ld_wait();
         } else {
-#pragma unroll
-          for (int i = 0; i < 32; i += 4) {
-            float f[4] = {0.f, 0.f, 0.f, 0.f};
-            if (begin != nullptr && ch * 32 + i < p.dv) load4(begin + ch * 32 + i, f);
-#pragma unroll
-            for (int j = 0; j < 4; ++j) v[i + j] = __float_as_uint(f[j]);
-          }
+          load_state_piece(begin, v, quarter * 32, ch * 32, p.dk, p.dv);
         }
         uint8_t* x = sX + (ch >> 1) * kPanelBytes;
         uint8_t* y = sY + (ch >> 1) * kPanelBytes;
@@ -584,7 +619,7 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
       ok = mbar_wait(&v_full[st], (c >> 1) & 1) && mbar_wait(t_done, ph);
       if (!ok) break;
       const float w = r < count && tok + r >= start ? pw[count - 1 - r] : 0.f;
-      for (int j = 0; j < p.v_panels; ++j) scale_panel_row(sV + st * kTile + j * kPanelBytes, sX + j * kPanelBytes, sY + j * kPanelBytes, r, w);
+      if (part < p.v_panels) scale_panel_row(sV + st * kTile + part * kPanelBytes, sX + part * kPanelBytes, sY + part * kPanelBytes, r, w);
       fence_proxy_async_smem();
       __syncwarp();
       if (lane == 0) mbar_arrive(vs_full);
@@ -592,18 +627,13 @@ lightning_run_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
     if (ok && !*abort_flag) ok = mbar_wait(h_done, (n - 1) & 1);
     if (ok && !*abort_flag && p.state != nullptr && run + 1 == p.runs) {
       tc_fence_after();
-      float* dst = p.state + ((static_cast<long long>(bi) * p.heads + h) * p.dk + r) * p.dv;
+      float* dst = p.state + (static_cast<long long>(bi) * p.heads + h) * p.dk * p.dv;
 #pragma unroll 1
-      for (int ch = 0; ch < p.v_panels * 2; ++ch) {
+      for (int ch = first_ch; ch < last_ch; ++ch) {
         uint32_t v[32];
         tmem_ld_32x32(tH + lane_sel + ch * 32, v);
         tmem_ld_wait();
-        if (r < p.dk) {
-#pragma unroll
-          for (int i = 0; i < 32; i += 4)
-            if (ch * 32 + i < p.dv)
-              *reinterpret_cast<float4*>(dst + ch * 32 + i) = make_float4(__uint_as_float(v[i]), __uint_as_float(v[i + 1]), __uint_as_float(v[i + 2]), __uint_as_float(v[i + 3]));
-        }
+        store_state_piece(dst, v, quarter * 32, ch * 32, p.dk, p.dv);
       }
     }
     if (!ok) fail(abort_flag, p.err, 255);
@@ -736,7 +766,7 @@ extern "C" int ttb_lightning_chunks(const void* q, long long ld_q, const void* k
     lightning_scan_kernel<<<dim3(static_cast<unsigned>((n / 4 + 255) / 256), heads, b), 256, 0, st>>>(work, before, chunk_powers, heads, p.runs, run_chunks, n);
   }
   TTB_COUNT_LAUNCH(1);
-  lightning_run_kernel<<<dim3(p.runs, heads, b), kChunkThreads, kRunSmem, st>>>(tq, tk, tv, p);
+  lightning_run_kernel<<<dim3(p.runs, heads, b), kRunThreads, kRunSmem, st>>>(tq, tk, tv, p);
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 

@@ -8,6 +8,7 @@
     python -m torchtune_b200.ops.microbench gate_up --tokens 8192 --dim 4096 --hidden 14336
     python -m torchtune_b200.ops.microbench comm --world 8 --numel 268435456             (peer-memory kernels, ranks emulated on one GPU)
     python -m torchtune_b200.ops.microbench latent --heads 16 --rank 512       (latent attention beside grouped-query attention)
+    python -m torchtune_b200.ops.microbench ragenex --heads 16 --streams 4     (lightning and span attention, stream steps)
     python -m torchtune_b200.ops.microbench suite --tokens 8192      (norm, RoPE, SwiGLU, loss, embedding, LoRA, grouped GEMM, NF4, offload copies)
 
 Each command prints one JSON line: median milliseconds over ``--iters`` launches (an L2 flush
@@ -240,6 +241,101 @@ def bench_latent(args, flush):
             t = _time_captured(lambda i: lambda: linear(xq, wj[i % 8]), it, wj[0].numel() * 2.0)
             emit("linear_joined", t, rows=T, gbs=wj[0].numel() * 2.0 / t / 1e6)
     return {"op": "latent", "heads": H, "kernels": len(rows)}
+
+
+def bench_ragenex(args, flush):
+    """Kernels of a decoder of lightning and grouped-query attention layers on four 32-bit streams beside the like kernels of other decoders
+    of equal width, heads and context: one JSON line per kernel."""
+    from . import clamped_glu, latent, recurrent, rms_norm, span, stream_step, swiglu
+    from ._cuda_attention import attention
+    from .mask import AttentionMask
+
+    H, d, D, S = args.heads, args.head_dim, args.dim, args.streams
+    G = max(1, H // 4)
+    bf = dict(device="cuda", dtype=torch.bfloat16)
+    it, wu = args.iters, args.warmup
+    decay = [1.0 - 2.0 ** -(1 + 10 * h / H) for h in range(H)]
+    rows = []
+
+    def emit(op, ms, **kw):
+        row = {"op": op, "ms": round(ms, 5), **{k: (round(v, 1) if isinstance(v, float) else v) for k, v in kw.items()}}
+        rows.append(row)
+        print(json.dumps(row), flush=True)
+
+    def copies(nbytes):
+        return int(max(4, min(64, 400e6 // nbytes + 1)))
+
+    with torch.no_grad():
+        for b, s in ((1, args.seq), (4, args.seq // 4)):
+            q, k, v = torch.randn(b * s, H * d, **bf), torch.randn(b, s, G, d, **bf), torch.randn(b, s, G, d, **bf)
+            pairs = b * H * s * (s + 1) / 2
+            t = _time(lambda: span.prefill(q, k, v, b=b, s=s, sk=s, slot0=0, heads=H, scale=0.07, bounds=latent.Bounds()), it, wu, flush)
+            emit("span_prefill", t, batch=b, seq=s, tflops=4 * pairs * d / t / 1e9)
+            t = _time(lambda: attention(q.view(b, s, H, d), k, v, AttentionMask(causal=True), None, 0.0), it, wu, flush)
+            emit("gqa_prefill", t, batch=b, seq=s, tflops=4 * pairs * d / t / 1e9)
+            qkv = torch.randn(b * s, 3 * H * d, **bf) * 0.5
+            q, k, v = qkv.split(H * d, dim=1)
+            state = torch.zeros(b, H, d, d, device="cuda")
+            run = lambda: recurrent.lightning(q, k, v, decay, state, b=b, s=s, heads=H, dim=d, vdim=d, fresh=True, starts=None, first=0)  # noqa: E731
+            silu, recurrent._silu = recurrent._silu, lambda *a: None
+            t = _time(run, it, wu, flush)
+            recurrent._silu = silu
+            nbytes = b * s * H * d * 8.0
+            emit("lightning_chunks", t, batch=b, seq=s, gbs=nbytes / t / 1e6)
+            t = _time(lambda: recurrent._silu(q, k, v), it, wu, flush)
+            emit("silu_rows", t, rows=b * s, gbs=b * s * H * d * 12.0 / t / 1e6)
+            o, gain, gate = torch.randn(b * s, H * d, **bf), torch.randn(H * d, **bf), torch.randn(b * s, H * d, **bf)
+            t = _time(lambda: recurrent.gated_norm(o, gain, gate, 1e-6), it, wu, flush)
+            emit("gated_norm", t, rows=b * s, gbs=b * s * H * d * 6.0 / t / 1e6)
+        for b, keys in ((1, 8192), (8, 4096), (32, 4096), (128, 2048)):
+            nbytes = b * keys * G * d * 4.0
+            n = copies(nbytes)
+            ks, vs = [torch.randn(b, keys, G, d, **bf) for _ in range(n)], [torch.randn(b, keys, G, d, **bf) for _ in range(n)]
+            q = torch.randn(b, H, d, **bf)
+            t = _time_captured(lambda i: lambda: span.decode(q, ks[i % n], vs[i % n], scale=0.07, slot=None, slot_host=keys - 1, bounds=latent.Bounds(), keys_visible=keys), it, nbytes)
+            emit("span_decode", t, batch=b, keys=keys, gbs=nbytes / t / 1e6)
+            m = AttentionMask(causal=False, bool_mask=torch.ones(b, 1, keys, dtype=torch.bool, device="cuda"))
+            t = _time_captured(lambda i: lambda: attention(q.view(b, 1, H, d), ks[i % n], vs[i % n], m, None, 0.0), it, nbytes)
+            emit("gqa_decode", t, batch=b, keys=keys, gbs=nbytes / t / 1e6)
+            del ks, vs
+            nbytes = b * H * d * d * 8.0
+            n = copies(nbytes)
+            states = [torch.zeros(b, H, d, d, device="cuda") for _ in range(n)]
+            x = [torch.randn(b, H * d, **bf) for _ in range(3)]
+            t = _time_captured(lambda i: lambda: recurrent.lightning(*x, decay, states[i % n], b=b, s=1, heads=H, dim=d, vdim=d, fresh=False, starts=None, first=9), it, nbytes)
+            emit("lightning_decode", t, batch=b, gbs=nbytes / t / 1e6)
+            del states
+        for T in (1, 16, 64, args.seq):
+            small = T < 1024
+            time = (lambda fn, nbytes: _time_captured(lambda i: fn, it, nbytes)) if small else (lambda fn, nbytes: _time(fn, it, wu, flush))
+            x, y, w = torch.randn(T, S, D, device="cuda"), torch.randn(T, D, **bf), torch.randn(D, **bf)
+            mix, c = torch.randn(S, S, **bf), torch.randn(S, **bf)
+            nbytes = T * D * (8.0 * S + 4)
+            t = time(lambda: stream_step(x, y, w, mix, c, c, w, eps=1e-6, centered=True), nbytes)
+            emit("stream_step", t, rows=T, gbs=nbytes / t / 1e6)
+            x1 = torch.randn(T, D, device="cuda")
+            t = time(lambda: latent.residual_norm(x1, y, w, w, 1e-6, 0.5, 1.0), T * D * 12.0)
+            emit("residual_norm", t, rows=T, gbs=T * D * 12.0 / t / 1e6)
+            t = time(lambda: rms_norm(y, w, 1e-6), T * D * 4.0)
+            emit("rms_norm", t, rows=T, gbs=T * D * 4.0 / t / 1e6)
+            packed = torch.randn(T, (H + 2 * G) * d, **bf)
+            q, k, v = packed.split([H * d, G * d, G * d], dim=1)
+            kc, vc = torch.zeros(1 if not small else T, T if not small else 8, G, d, **bf), torch.zeros(1 if not small else T, T if not small else 8, G, d, **bf)
+            gq, gk = torch.randn(H * d, **bf), torch.randn(G * d, **bf)
+            run = lambda: span.prepare(q, k, v, gq, gk, kc, vc, None, s=1 if small else T, slot=None, slot_host=0, eps=1e-6, coef=0.1, every=512)  # noqa: E731
+            nbytes = packed.numel() * 4.0
+            emit("span_prepare", t := time(run, nbytes), rows=T, gbs=nbytes / t / 1e6)
+            g, u = torch.randn(T, 4 * D, **bf), torch.randn(T, 4 * D, **bf)
+            nbytes = T * D * 24.0
+            emit("clamped_glu", t := time(lambda: clamped_glu(g, u, 7.0, 1.702), nbytes), rows=T, gbs=nbytes / t / 1e6)
+            emit("swiglu", t := time(lambda: swiglu(g, u), nbytes), rows=T, gbs=nbytes / t / 1e6)
+        from ._cuda import gate_up_swiglu
+
+        x, w1, w3 = torch.randn(args.seq, D, **bf), torch.randn(4 * D, D, **bf) * D**-0.5, torch.randn(4 * D, D, **bf) * D**-0.5
+        for op, clamp in (("gemm_clamped_glu", (7.0, 1.702)), ("gemm_swiglu", None)):
+            t = _time(lambda: gate_up_swiglu(x, w1, w3, clamp), it, wu, flush)
+            emit(op, t, rows=args.seq, tflops=2.0 * args.seq * D * 8 * D / t / 1e9)
+    return {"op": "ragenex", "heads": H, "kernels": len(rows)}
 
 
 def bench_rmsnorm(args, flush):
@@ -559,13 +655,19 @@ def main() -> None:
     la.add_argument("--rank", type=int, default=512)
     la.add_argument("--dim", type=int, default=2048)
     la.add_argument("--seq", type=int, default=8192)
+    rx = sub.add_parser("ragenex")
+    rx.add_argument("--heads", type=int, default=16)
+    rx.add_argument("--head-dim", type=int, default=128)
+    rx.add_argument("--dim", type=int, default=2048)
+    rx.add_argument("--streams", type=int, default=4)
+    rx.add_argument("--seq", type=int, default=8192)
     su = sub.add_parser("suite")
     su.add_argument("--tokens", type=int, default=8192)
     args = ap.parse_args()
     from ._lib import check_device_errors
 
     flush = torch.empty(256 << 20, dtype=torch.uint8, device="cuda")
-    fn = {"gemm": bench_gemm, "gemm_fp8": bench_gemm_fp8, "gemm_mxfp8": bench_gemm_mxfp8, "attention": bench_attention, "rmsnorm": bench_rmsnorm, "adamw": bench_adamw, "adamw8bit": bench_adamw8bit, "gate_up": bench_gate_up, "comm": bench_comm, "latent": bench_latent, "suite": bench_suite}[args.op]
+    fn = {"gemm": bench_gemm, "gemm_fp8": bench_gemm_fp8, "gemm_mxfp8": bench_gemm_mxfp8, "attention": bench_attention, "rmsnorm": bench_rmsnorm, "adamw": bench_adamw, "adamw8bit": bench_adamw8bit, "gate_up": bench_gate_up, "comm": bench_comm, "latent": bench_latent, "ragenex": bench_ragenex, "suite": bench_suite}[args.op]
     res = fn(args, flush)
     check_device_errors()
     print(json.dumps(res), flush=True)
