@@ -453,6 +453,20 @@ def test_model(tmp_path, name, dtype, tol):
     _errors()
 
 
+@pytest.mark.parametrize("dtype,tol", [(F32, 5e-5), (BF16, 8e-2)])
+def test_long_decoding(tmp_path, dtype, tol):
+    """Far more decoded tokens than the prompt has, over several key tiles, replayed as one graph."""
+    from torchtune_b200.generation import BatchDecoder
+
+    cfg, w, model = _load(tmp_path, "plain", dtype)
+    s = np.random.default_rng(5).integers(0, cfg["vocab"], 290).tolist()
+    with torch.inference_mode():
+        dec = BatchDecoder(model, torch.device(DEV), dtype, 290)
+        h = [dec.begin([s[:2]])[0]] + [dec.advance([t])[0] for t in s[2:]]
+        assert _rms_error(dec.logits(torch.cat(h)), oracle.forward(cfg, w, s)) < tol
+    _errors()
+
+
 def test_greedy_generation_matches(tmp_path):
     """fp32 generation through ``generate`` picks the oracle's tokens, alone and in a padded batch (decode steps are a replayed graph)."""
     from torchtune_b200.generation import generate

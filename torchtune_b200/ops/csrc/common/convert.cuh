@@ -75,6 +75,26 @@ __device__ __forceinline__ float logistic(float z) {
   else return 1.f / (1.f + __expf(-z));
 }
 
+// Sums of two values over all threads of a CTA; every thread gets them.
+template <int THREADS>
+__device__ __forceinline__ float2 cta_sum2(float a, float b, float2* scratch) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    a += __shfl_xor_sync(0xffffffffu, a, o);
+    b += __shfl_xor_sync(0xffffffffu, b, o);
+  }
+  const int w = threadIdx.x >> 5, l = threadIdx.x & 31;
+  if (l == 0) scratch[w] = make_float2(a, b);
+  __syncthreads();
+  float2 t = make_float2(0.f, 0.f);
+#pragma unroll
+  for (int i = 0; i < THREADS / 32; ++i) {
+    const float2 v = scratch[i];
+    t.x += v.x, t.y += v.y;
+  }
+  return t;
+}
+
 // Sum over all threads of a CTA; every thread gets it.
 template <int THREADS>
 __device__ __forceinline__ float cta_sum(float v, float* scratch) {

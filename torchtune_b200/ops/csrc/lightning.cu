@@ -666,39 +666,48 @@ __global__ void __launch_bounds__(256) silu_rows_kernel(bf16* __restrict__ x, lo
   }
 }
 
-template <typename O, typename T, bool VEC>
+// V > 0: width % 4 == 0 and width <= 1024 * V, the row waits in registers for its sum of squares.  V == 0: any width, the row is read again.
+template <typename O, typename T, int V>
 __global__ void __launch_bounds__(256) gated_norm_kernel(const O* __restrict__ o, const T* __restrict__ gain, const T* __restrict__ gate, long long ld_gate, T* __restrict__ out,
                                                          int width, float eps) {
   __shared__ float scratch[8];
   const long long row = blockIdx.x;
   const O* src = o + row * width;
   const T* g = gate + row * ld_gate;
+  const float inv = 1.f / static_cast<float>(width);
   float ss = 0.f;
-  if constexpr (VEC) {
-    for (int i = threadIdx.x * 4; i < width; i += 1024) {
-      float f[4];
-      load4(src + i, f);
+  if constexpr (V > 0) {
+    float f[V][4], z[V][4];
 #pragma unroll
-      for (int j = 0; j < 4; ++j) ss += f[j] * f[j];
+    for (int k = 0; k < V; ++k) {
+      const int i = (threadIdx.x + k * 256) * 4;
+      f[k][0] = f[k][1] = f[k][2] = f[k][3] = 0.f;
+      if (i < width) {
+        load4(src + i, f[k]);
+        load4(g + i, z[k]);
+      }
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss += f[k][j] * f[k][j];
+    const float rs = 1.f / sqrtf(cta_sum<256>(ss, scratch) * inv + eps);
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      const int i = (threadIdx.x + k * 256) * 4;
+      if (i >= width) continue;
+      float w[4];
+      load4(gain + i, w);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) w[j] = f[k][j] * rs * w[j] * logistic<T>(z[k][j]);
+      store4(out + row * width + i, w);
     }
   } else {
     for (int i = threadIdx.x; i < width; i += 256) {
       const float f = as_float(src[i]);
       ss += f * f;
     }
-  }
-  const float rs = 1.f / sqrtf(cta_sum<256>(ss, scratch) / static_cast<float>(width) + eps);
-  if constexpr (VEC) {
-    for (int i = threadIdx.x * 4; i < width; i += 1024) {
-      float f[4], w[4], z[4];
-      load4(src + i, f);
-      load4(gain + i, w);
-      load4(g + i, z);
-#pragma unroll
-      for (int j = 0; j < 4; ++j) f[j] = f[j] * rs * w[j] * logistic<T>(z[j]);
-      store4(out + row * width + i, f);
-    }
-  } else {
+    const float rs = 1.f / sqrtf(cta_sum<256>(ss, scratch) * inv + eps);
     for (int i = threadIdx.x; i < width; i += 256) out[row * width + i] = float_as<T>(as_float(src[i]) * rs * as_float(gain[i]) * logistic<T>(as_float(g[i])));
   }
 }
@@ -708,12 +717,15 @@ static int launch_gated_norm(const void* o, const void* gain, const void* gate, 
   const bool vec = width % 4 == 0 && ld_gate % 4 == 0 &&
                    !((reinterpret_cast<uintptr_t>(o) | reinterpret_cast<uintptr_t>(gain) | reinterpret_cast<uintptr_t>(gate) | reinterpret_cast<uintptr_t>(out)) & 15);
   TTB_COUNT_LAUNCH(1);
-  if (vec)
-    gated_norm_kernel<O, T, true><<<static_cast<unsigned>(rows), 256, 0, st>>>(static_cast<const O*>(o), static_cast<const T*>(gain), static_cast<const T*>(gate), ld_gate,
-                                                                               static_cast<T*>(out), width, eps);
-  else
-    gated_norm_kernel<O, T, false><<<static_cast<unsigned>(rows), 256, 0, st>>>(static_cast<const O*>(o), static_cast<const T*>(gain), static_cast<const T*>(gate), ld_gate,
-                                                                                static_cast<T*>(out), width, eps);
+#define TTB_GATED_NORM(V)                                                                                                                                                        \
+  gated_norm_kernel<O, T, V><<<static_cast<unsigned>(rows), 256, 0, st>>>(static_cast<const O*>(o), static_cast<const T*>(gain), static_cast<const T*>(gate), ld_gate, \
+                                                                          static_cast<T*>(out), width, eps)
+  if (!vec || width > 8192) TTB_GATED_NORM(0);
+  else if (width <= 1024) TTB_GATED_NORM(1);
+  else if (width <= 2048) TTB_GATED_NORM(2);
+  else if (width <= 4096) TTB_GATED_NORM(4);
+  else TTB_GATED_NORM(8);
+#undef TTB_GATED_NORM
   return cudaGetLastError() == cudaSuccess ? kOk : kErrDriver;
 }
 

@@ -24,71 +24,99 @@ struct PrepareParams {
 static constexpr int kThreads = 256;
 
 template <typename T, int W>
-struct Pack;  // W consecutive elements as fp32
+struct Pack;  // W consecutive elements
 template <typename T>
 struct Pack<T, 1> {
-  static __device__ __forceinline__ void load(const T* p, float (&f)[1]) { f[0] = as_float(*p); }
-  static __device__ __forceinline__ void store(T* p, const float (&f)[1]) { *p = float_as<T>(f[0]); }
+  using Raw = T;
+  static __device__ __forceinline__ Raw zero() { return float_as<T>(0.f); }
+  static __device__ __forceinline__ void unpack(const Raw& r, float (&f)[1]) { f[0] = as_float(r); }
+  static __device__ __forceinline__ Raw pack(const float (&f)[1]) { return float_as<T>(f[0]); }
 };
 template <>
 struct Pack<__nv_bfloat16, 8> {
-  static __device__ __forceinline__ void load(const __nv_bfloat16* p, float (&f)[8]) { unpack_bf16x8(*reinterpret_cast<const uint4*>(p), f); }
-  static __device__ __forceinline__ void store(__nv_bfloat16* p, const float (&f)[8]) { *reinterpret_cast<uint4*>(p) = pack_bf16x8(f); }
+  using Raw = uint4;
+  static __device__ __forceinline__ Raw zero() { return make_uint4(0u, 0u, 0u, 0u); }
+  static __device__ __forceinline__ void unpack(const Raw& r, float (&f)[8]) { unpack_bf16x8(r, f); }
+  static __device__ __forceinline__ Raw pack(const float (&f)[8]) { return pack_bf16x8(f); }
+};
+
+// A thread's pieces of a row: the first HELD of them wait in registers between the sum of squares and the scaling, the rest (of a very
+// wide row) are read again.
+template <typename T, int W, int HELD>
+struct Row {
+  using P = Pack<T, W>;
+  using Raw = typename P::Raw;
+  Raw r[HELD];
+  static __device__ __forceinline__ int at(int k) { return (threadIdx.x + k * kThreads) * W; }
+  static __device__ __forceinline__ const Raw& raw(const T* p) { return *reinterpret_cast<const Raw*>(p); }
+  static __device__ __forceinline__ float squares_of(const Raw& v) {
+    float f[W], ss = 0.f;
+    P::unpack(v, f);
+#pragma unroll
+    for (int j = 0; j < W; ++j) ss += f[j] * f[j];
+    return ss;
+  }
+  static __device__ __forceinline__ Raw scaled(const Raw& v, const T* gain, float by) {
+    float f[W], g[W];
+    P::unpack(v, f);
+    if (gain != nullptr) P::unpack(raw(gain), g);
+#pragma unroll
+    for (int j = 0; j < W; ++j) f[j] = f[j] * by * (gain != nullptr ? g[j] : 1.f);
+    return P::pack(f);
+  }
+  __device__ __forceinline__ void load(const T* p, int n) {
+#pragma unroll
+    for (int k = 0; k < HELD; ++k) r[k] = at(k) < n ? raw(p + at(k)) : P::zero();
+  }
+  __device__ __forceinline__ float squares(const T* p, int n) const {
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < HELD; ++k) ss += squares_of(r[k]);
+    for (int i = at(HELD); i < n; i += kThreads * W) ss += squares_of(raw(p + i));
+    return ss;
+  }
+  __device__ __forceinline__ void store(T* dst, const T* p, const T* gain, int n, float by) const {
+#pragma unroll
+    for (int k = 0; k < HELD; ++k)
+      if (at(k) < n) *reinterpret_cast<Raw*>(dst + at(k)) = scaled(r[k], gain != nullptr ? gain + at(k) : nullptr, by);
+    for (int i = at(HELD); i < n; i += kThreads * W) *reinterpret_cast<Raw*>(dst + i) = scaled(raw(p + i), gain != nullptr ? gain + i : nullptr, by);
+  }
 };
 
 template <typename T, int W>
-__device__ __forceinline__ float squares(const T* p, int n) {
-  float ss = 0.f;
-  for (int i = threadIdx.x * W; i < n; i += kThreads * W) {
-    float f[W];
-    Pack<T, W>::load(p + i, f);
-#pragma unroll
-    for (int j = 0; j < W; ++j) ss += f[j] * f[j];
-  }
-  return ss;
-}
-
-template <typename T, int W>
-__device__ __forceinline__ void scaled(T* dst, const T* src, const T* gain, int n, float by) {
-  for (int i = threadIdx.x * W; i < n; i += kThreads * W) {
-    float f[W], g[W];
-    Pack<T, W>::load(src + i, f);
-    if (gain != nullptr) Pack<T, W>::load(gain + i, g);
-#pragma unroll
-    for (int j = 0; j < W; ++j) f[j] = f[j] * by * (gain != nullptr ? g[j] : 1.f);
-    Pack<T, W>::store(dst + i, f);
-  }
-}
-
-template <typename T, int W>
 __global__ void __launch_bounds__(kThreads) span_prepare_kernel(const PrepareParams p) {
-  __shared__ float scratch[kThreads / 32];
+  __shared__ float2 scratch[kThreads / 32];
   const long long row = blockIdx.x;
   const int bi = static_cast<int>(row / p.s), i = static_cast<int>(row % p.s);
-  const int slot = (p.slot != nullptr ? *p.slot : p.slot_host) + i;
   T* q = static_cast<T*>(p.q) + row * p.ld_q;
   const T* k = static_cast<const T*>(p.k) + row * p.ld_k;
   const T* v = static_cast<const T*>(p.v) + row * p.ld_v;
   const T* q_gain = static_cast<const T*>(p.q_gain);
   const T* k_gain = static_cast<const T*>(p.k_gain);
+  Row<T, W, 2> rq;
+  Row<T, W, 1> rk, rv;
+  rq.load(q, p.q_width);
+  rk.load(k, p.k_width);
+  rv.load(v, p.v_width);
+  const int slot = (p.slot != nullptr ? *p.slot : p.slot_host) + i;
   float by_q = 1.f, by_k = 1.f;
   if (q_gain != nullptr) {
-    const float sq = squares<T, W>(q, p.q_width), sk = squares<T, W>(k, p.k_width);
-    by_q = 1.f / sqrtf(cta_sum<kThreads>(sq, scratch) / static_cast<float>(p.q_width) + p.eps);
-    by_k = 1.f / sqrtf(cta_sum<kThreads>(sk, scratch) / static_cast<float>(p.k_width) + p.eps);
+    const float2 ss = cta_sum2<kThreads>(rq.squares(q, p.q_width), rk.squares(k, p.k_width), scratch);
+    by_q = 1.f / sqrtf(ss.x / static_cast<float>(p.q_width) + p.eps);
+    by_k = 1.f / sqrtf(ss.y / static_cast<float>(p.k_width) + p.eps);
   }
   if (p.coef != 0.f) {
     const int pos = max(p.pos != nullptr ? p.pos[row] : slot, 0);
     by_q *= 1.f + p.coef * logf(static_cast<float>((pos + 1) / p.every + 1));
   }
-  if (q_gain != nullptr || p.coef != 0.f) scaled<T, W>(q, q, q_gain, p.q_width, by_q);
+  if (q_gain != nullptr || p.coef != 0.f) rq.store(q, q, q_gain, p.q_width, by_q);
   if (slot < 0 || slot >= p.slots) {
     if (threadIdx.x == 0) TTB_NOTE_VIOLATION(span);
     return;
   }
   const long long at = static_cast<long long>(bi) * p.slots + slot;
-  scaled<T, W>(static_cast<T*>(p.keys) + at * p.k_width, k, k_gain, p.k_width, by_k);
-  scaled<T, W>(static_cast<T*>(p.values) + at * p.v_width, v, static_cast<const T*>(nullptr), p.v_width, 1.f);
+  rk.store(static_cast<T*>(p.keys) + at * p.k_width, k, k_gain, p.k_width, by_k);
+  rv.store(static_cast<T*>(p.values) + at * p.v_width, v, nullptr, p.v_width, 1.f);
 }
 
 }  // namespace span
